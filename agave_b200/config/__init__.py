@@ -1,7 +1,8 @@
 from .base import (AttentionSpec, BlockSpec, ConfigError, DenseFeedForwardSpec, DistanceBiasSpec,
                    GatedFeedForwardSpec, IdentityNormSpec, LatentAttentionSpec, LayerCall,
-                   LayerNormSpec, ModelSpec, NormSpec, QueryTemperatureSpec,
-                   RoutedFeedForwardSpec, RotarySpec, WavelengthScalingSpec, default_schedule)
+                   LayerNormSpec, ModelSpec, NormSpec, ParallelBlockSpec, QueryTemperatureSpec,
+                   RoutedFeedForwardSpec, RotarySpec, SelectiveScanSpec, SideBySideSpec,
+                   StateSpaceSpec, WavelengthScalingSpec, default_schedule)
 from .registry import (load_config, read_config_json, register_architecture,
                        registered_architectures, resolve_architecture)
 from .gemma3 import Gemma3Config
@@ -9,6 +10,7 @@ from .ramilorn import RamilornConfig
 from .zazerax import ZazeraxConfig
 from .bovozen import BovozenConfig
 from .kadavik import KadavikConfig
+from .savovik import SavovikConfig
 
 __all__ = [
     "AttentionSpec", "BlockSpec", "ConfigError", "GatedFeedForwardSpec", "LayerCall",
@@ -16,6 +18,7 @@ __all__ = [
     "RotarySpec", "RamilornConfig", "default_schedule", "load_config",
     "read_config_json", "register_architecture", "registered_architectures",
     "resolve_architecture", "Gemma3Config", "ZazeraxConfig", "DenseFeedForwardSpec",
-    "DistanceBiasSpec", "IdentityNormSpec", "LatentAttentionSpec", "WavelengthScalingSpec",
-    "BovozenConfig", "KadavikConfig",
+    "DistanceBiasSpec", "ParallelBlockSpec", "SelectiveScanSpec", "SideBySideSpec",
+    "StateSpaceSpec", "IdentityNormSpec", "LatentAttentionSpec", "WavelengthScalingSpec",
+    "BovozenConfig", "KadavikConfig", "SavovikConfig",
 ]

@@ -180,6 +180,13 @@ class AttentionSpec:
     # the cache keeps every key of this layer whatever its own mask: another call reads the
     # entry through a mask that reaches further back
     keep_all_keys: bool = False
+    # biases added to the q, k and v projections (tensors ``q_proj.bias`` ...), before any norm
+    qkv_bias: bool = False
+    # scaled scores become softcap * tanh(score / softcap) before the mask; None: no cap
+    softcap: Optional[float] = None
+    # every value head is divided by its root mean square (this eps under the root, no weight)
+    # before it is cached; None: values stay as projected
+    value_norm_eps: Optional[float] = None
 
     @property
     def v_dim(self) -> int:
@@ -253,6 +260,55 @@ class MatrixMemorySpec:
     gate_cap: float = 15.0
     eps: float = 1e-6
     den_eps: float = 1e-6
+
+
+@dataclass(frozen=True)
+class SelectiveScanSpec:
+    """A recurrent mixer: the selective scan of Mamba, a decay per channel, state and token.
+
+    W_in x = [u | z], ``inner`` wide each.  u passes a causal convolution over ``conv_taps``
+    tokens per channel (with a bias) and silu.  W_x u = [r | B | C] (``dt_rank``, ``state`` and
+    ``state`` wide); dt = softplus(W_dt r + b_dt) per channel.  Per channel c and state n, with
+    A = -exp(A_log):  S[c, n] <- exp(dt_c A[c, n]) S[c, n] + dt_c u_c B_n;  y_c = sum_n S[c, n]
+    C_n + D_c u_c.  y * silu(z) feeds the output product.  S (32-bit) and the convolution's last
+    conv_taps - 1 inputs are a fixed size per sequence."""
+    kind: str = "selective_scan"
+    inner: int = 0
+    state: int = 0
+    dt_rank: int = 0
+    conv_taps: int = 1
+
+
+@dataclass(frozen=True)
+class StateSpaceSpec:
+    """A recurrent mixer: the state-space form of Mamba-2, one decay per head and token.
+
+    W_in x = [z | u | B | C | dt] (H dv, H dv, G N, G N and H wide, H = ``n_heads``, dv =
+    ``value_dim``, G = ``n_groups``, N = ``state``).  u, B and C together pass a causal
+    convolution over ``conv_taps`` tokens per channel (with a bias) and silu;
+    dt <- softplus(dt + dt_bias).  Head h uses group h // (H / G):
+    S <- exp(-exp(A_log_h) dt) S + dt B u^T (S is N x dv);  y = S^T C + D_h u.  y * silu(z) is
+    divided, in ``norm_groups`` equal parts, by each part's root mean square (``eps``), times a
+    weight per channel, and goes through the output product.  S (32-bit) and the convolution's
+    last conv_taps - 1 inputs are a fixed size per sequence."""
+    kind: str = "state_space"
+    n_heads: int = 0
+    value_dim: int = 0
+    state: int = 0
+    n_groups: int = 1
+    norm_groups: int = 1
+    conv_taps: int = 1
+    eps: float = 1e-6
+
+
+@dataclass(frozen=True)
+class SideBySideSpec:
+    """Two mixers that read the same input: left_scale * left + right_scale * right."""
+    kind: str = "side_by_side"
+    left: object = None
+    right: object = None
+    left_scale: float = 1.0
+    right_scale: float = 1.0
 
 
 @dataclass(frozen=True)
@@ -347,6 +403,21 @@ class BlockSpec:
     residual_mult: float = 1.0
     # a per-layer input from the token, added after the feed-forward (None: none)
     token_side: Optional[TokenSideSpec] = None
+
+
+@dataclass(frozen=True)
+class ParallelBlockSpec:
+    """One layer whose branches read one norm: with x = norm(h),
+    h += gate_m(x) * mixer(x) + gate_f(x) * ffn(x).
+
+    ``gated``: gate_m(x) = sigmoid(W x + b) element by element (tensors ``mixer_gate.weight``,
+    ``mixer_gate.bias``), gate_f likewise (``ffn_gate.*``); else both are one.
+    ``feed_forward`` None: the layer has no feed-forward branch."""
+    mixer: object = None
+    feed_forward: object = None
+    norm: object = NormSpec()
+    gated: bool = False
+    kind: str = "parallel"
 
 
 @dataclass(frozen=True)

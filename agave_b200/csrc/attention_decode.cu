@@ -77,13 +77,13 @@ __device__ __forceinline__ float2 load_pair(const __nv_bfloat16* p) {
 struct DecodeArgs {
     const void* q;             // [B, nh, hd] rows of stride q_stride
     long long q_stride;
-    void* out;                 // [B, nh * hd]
+    void* out;                 // [B, nh * hdv]
     const void* k_pool;        // [n_pages, page, nkv, hd] of this layer
-    const void* v_pool;
+    const void* v_pool;        // [n_pages, page, nkv, hdv]
     const int* page_table;     // [n_slots, max_pages]
     const int* slots;          // [B]; negative = padding entry
     const int* positions;      // [B] position of the query (its key is stored already)
-    float* part_acc;           // [B, nh, S, hd]
+    float* part_acc;           // [B, nh, S, hdv]
     float* part_ml;            // [B, nh, S, 2]
     int* counters;             // [B * gridDim.y], zero before and after a launch
     int max_pages, page, cap, nh, nkv, hd, window, n_splits, chunk;
@@ -95,6 +95,10 @@ struct DecodeArgs {
     // walk over the keys then starts min(keep_first, window start) places before the window:
     // those places stand for the first keys (see walked_key).  Copied tiles only.
     int keep_first = 0;
+    float softcap = 0.f;       // > 0: the scaled score s becomes softcap * tanh(s / softcap)
+    // The value head size (out and part_acc are hdv wide a head).  Where it is not hd the tiles
+    // come by copies and nothing is fused.
+    int hdv = 0;
 };
 
 // The walk's first place for a query at position p whose window starts at lo_w, and the key a
@@ -109,6 +113,11 @@ __device__ __forceinline__ int walked_key(int place, int lo, int lo_w) {
 // The learned bias of head h for the key at position j seen from position p.
 __device__ __forceinline__ float distance_bias(const DecodeArgs& a, int p, int j, int h) {
     return a.dist_bias[(size_t)h * a.n_dist + min(p - j, a.n_dist - 1)];
+}
+
+// The scaled score under the soft cap, if there is one.
+__device__ __forceinline__ float capped(const DecodeArgs& a, float s) {
+    return a.softcap > 0.f ? soft_capped_ex2(s, 2.0f * 1.4426950408889634f / a.softcap, a.softcap) : s;
 }
 
 // What the sink of head h adds to a normaliser taken relative to the maximum m.
@@ -151,7 +160,7 @@ __device__ __forceinline__ void finish_split(const DecodeArgs& a, int b, int h0,
                                              bool write_ml = true) {
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int nthreads = blockDim.x, nwarps = nthreads >> 5;
-    const int hd = a.hd;
+    const int hd = a.hdv;                      // (values only from here on)
     if (arrivals == 0) arrivals = used;        // one arrival per partial result
     if (write_ml && tid < gc) {
         float* dst = a.part_ml + (((size_t)b * a.nh + h0 + tid) * a.n_splits + split) * 2;
@@ -247,13 +256,13 @@ attention_decode_split_kernel(DecodeArgs a) {
     const int g = blockIdx.y / chunks_per_group;              // kv head
     const int h0 = g * G + (blockIdx.y % chunks_per_group) * AD_GC;   // first query head
     const int gc = min(AD_GC, g * G + G - h0);                // heads handled here
-    const int hd = a.hd, CH = a.chunk;
+    const int hd = a.hd, hdv = a.hdv, CH = a.chunk;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    T* outp = (T*)a.out + ((size_t)b * a.nh + h0) * hd;
+    T* outp = (T*)a.out + ((size_t)b * a.nh + h0) * hdv;
     const int slot = a.slots[b];
     if (slot < 0) {
         if (split == 0)
-            for (int i = tid; i < gc * hd; i += AD_THREADS) outp[i] = from_f32<T>(0.f);
+            for (int i = tid; i < gc * hdv; i += AD_THREADS) outp[i] = from_f32<T>(0.f);
         return;
     }
     const int p = a.positions[b];
@@ -266,7 +275,7 @@ attention_decode_split_kernel(DecodeArgs a) {
 
     T* Ks = reinterpret_cast<T*>(smem_raw);
     T* Vs = Ks + (size_t)CH * hd;
-    float* qs = reinterpret_cast<float*>(Vs + (size_t)CH * hd);   // [AD_GC][hd]
+    float* qs = reinterpret_cast<float*>(Vs + (size_t)CH * hdv);  // [AD_GC][hd]
     float* sc = qs + AD_GC * hd;                                  // [AD_GC][CH]
     float* stat = sc + AD_GC * CH;                                // [AD_GC][2]
     int* rowoff = reinterpret_cast<int*>(stat + AD_GC * 2);       // [CH] row index in the pool
@@ -290,7 +299,15 @@ attention_decode_split_kernel(DecodeArgs a) {
         const int r = i / vec_per_row, c = (i % vec_per_row) * VEC;
         const size_t off = ((size_t)rowoff[r] * a.nkv + g) * hd + c;
         cp_async16(Ks + (size_t)r * hd + c, (const T*)a.k_pool + off);
-        cp_async16(Vs + (size_t)r * hd + c, (const T*)a.v_pool + off);
+        if (hdv == hd) cp_async16(Vs + (size_t)r * hd + c, (const T*)a.v_pool + off);
+    }
+    if (hdv != hd) {
+        const int vec_per_v = hdv / VEC;
+        for (int i = tid; i < n * vec_per_v; i += AD_THREADS) {
+            const int r = i / vec_per_v, c = (i % vec_per_v) * VEC;
+            cp_async16(Vs + (size_t)r * hdv + c,
+                       (const T*)a.v_pool + ((size_t)rowoff[r] * a.nkv + g) * hdv + c);
+        }
     }
     cp_async_wait_all();
     __syncthreads();
@@ -317,6 +334,7 @@ attention_decode_split_kernel(DecodeArgs a) {
 #pragma unroll
         for (int hh = 0; hh < AD_GC; ++hh) {
             float t = warp_sum(s[hh]) * a.scale;
+            if (a.softcap > 0.f) t = soft_capped(t, a.softcap);
             if (a.dist_bias && hh < gc) t += distance_bias(a, p, j0 + r, h0 + hh);
             if (lane == 0 && hh < gc) sc[hh * CH + r] = t;
         }
@@ -341,10 +359,10 @@ attention_decode_split_kernel(DecodeArgs a) {
     }
     __syncthreads();
     // ---- weighted sum of the values: each thread owns pairs of output dimensions
-    for (int d = tid * 2; d < hd; d += AD_THREADS * 2) {
+    for (int d = tid * 2; d < hdv; d += AD_THREADS * 2) {
         float acc[AD_GC][2] = {};
         for (int r = 0; r < n; ++r) {
-            const float2 vv = load_pair(Vs + (size_t)r * hd + d);
+            const float2 vv = load_pair(Vs + (size_t)r * hdv + d);
 #pragma unroll
             for (int hh = 0; hh < AD_GC; ++hh) {
                 if (hh < gc) {
@@ -359,11 +377,11 @@ attention_decode_split_kernel(DecodeArgs a) {
             if (hh < gc) {
                 if (used == 1) {
                     const float inv = 1.0f / (stat[hh * 2 + 1] + sink_term(a, h0 + hh, stat[hh * 2]));
-                    outp[hh * hd + d] = from_f32<T>(acc[hh][0] * inv);
-                    outp[hh * hd + d + 1] = from_f32<T>(acc[hh][1] * inv);
+                    outp[hh * hdv + d] = from_f32<T>(acc[hh][0] * inv);
+                    outp[hh * hdv + d + 1] = from_f32<T>(acc[hh][1] * inv);
                 } else {
                     float* dst = a.part_acc +
-                                 (((size_t)b * a.nh + h0 + hh) * a.n_splits + split) * hd + d;
+                                 (((size_t)b * a.nh + h0 + hh) * a.n_splits + split) * hdv + d;
                     dst[0] = acc[hh][0];
                     dst[1] = acc[hh][1];
                 }
@@ -372,7 +390,7 @@ attention_decode_split_kernel(DecodeArgs a) {
     }
     if (used == 1) return;
     finish_split<T>(a, b, h0, gc, used, split, stat, reinterpret_cast<float*>(smem_raw),
-                    (int)(((size_t)2 * CH * hd * sizeof(T)) / sizeof(float)), &s_last, outp);
+                    (int)(((size_t)CH * (hd + hdv) * sizeof(T)) / sizeof(float)), &s_last, outp);
 }
 
 // ------------------------------------------------------- tensor-core variant
@@ -612,15 +630,15 @@ attention_decode_mma_kernel(DecodeArgs a, int cs, FuseQK fq,
     const int g = blockIdx.y / groups_per_kv;
     const int h0 = g * G + (blockIdx.y % groups_per_kv) * DM_HEADS;
     const int gc = min(DM_HEADS, g * G + G - h0);
-    const int hd = a.hd;
+    const int hd = a.hd, hdv = a.hdv;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int gid = lane >> 2, tig = lane & 3;
-    T* outp = (T*)a.out + ((size_t)b * a.nh + h0) * hd;
+    T* outp = (T*)a.out + ((size_t)b * a.nh + h0) * hdv;
     const int slot = a.slots[b];
     if (slot < 0) {
         pdl_wait();
         if (split == 0)
-            for (int i = tid; i < gc * hd; i += DM_THREADS) outp[i] = __float2bfloat16_rn(0.f);
+            for (int i = tid; i < gc * hdv; i += DM_THREADS) outp[i] = __float2bfloat16_rn(0.f);
         return;
     }
     const int p = a.positions[b];
@@ -752,14 +770,15 @@ attention_decode_mma_kernel(DecodeArgs a, int cs, FuseQK fq,
             const int r = i / CPR, c = i % CPR;
             const int off = dm_swz<HDP>(r, c);
             if (r == skip) continue;
-            if (ro[r] >= 0 && c * 8 < hd) {
-                const size_t src = ((size_t)ro[r] * a.nkv + g) * hd + c * 8;
-                cp_async16(kd + off, (const T*)a.k_pool + src);
-                cp_async16(vd + off, (const T*)a.v_pool + src);
-            } else {
+            const size_t head = (size_t)ro[r] * a.nkv + g;
+            if (ro[r] >= 0 && c * 8 < hd)
+                cp_async16(kd + off, (const T*)a.k_pool + head * hd + c * 8);
+            else
                 *reinterpret_cast<uint4*>(kd + off) = make_uint4(0, 0, 0, 0);
+            if (ro[r] >= 0 && c * 8 < hdv)
+                cp_async16(vd + off, (const T*)a.v_pool + head * hdv + c * 8);
+            else
                 *reinterpret_cast<uint4*>(vd + off) = make_uint4(0, 0, 0, 0);
-            }
         }
         cp_async_commit();
     };
@@ -838,14 +857,15 @@ attention_decode_mma_kernel(DecodeArgs a, int cs, FuseQK fq,
         }
         for (int c = tid; c < CPR; c += DM_THREADS) {
             const int off = kv_swz<HDP, TMA>(r, c);
-            if (cache_row >= 0 && c * 8 < hd) {
-                const size_t src = ((size_t)cache_row * a.nkv + g) * hd + c * 8;
-                cp_async16(Ks + off, (const T*)a.k_pool + src);
-                cp_async16(Vs + off, (const T*)a.v_pool + src);
-            } else {
+            const size_t head = (size_t)cache_row * a.nkv + g;
+            if (cache_row >= 0 && c * 8 < hd)
+                cp_async16(Ks + off, (const T*)a.k_pool + head * hd + c * 8);
+            else
                 *reinterpret_cast<uint4*>(Ks + off) = make_uint4(0, 0, 0, 0);
+            if (cache_row >= 0 && c * 8 < hdv)
+                cp_async16(Vs + off, (const T*)a.v_pool + head * hdv + c * 8);
+            else
                 *reinterpret_cast<uint4*>(Vs + off) = make_uint4(0, 0, 0, 0);
-            }
         }
     };
     if (!TMA && r_new >= 0 && r_new < DM_KEYS) new_row(Ks, Vs, r_new, rowoff[r_new]);
@@ -940,7 +960,7 @@ attention_decode_mma_kernel(DecodeArgs a, int cs, FuseQK fq,
             for (int e = 0; e < 4; ++e) {
                 const int key = warp * 16 + i * 8 + tig * 2 + (e & 1);
                 const int row = gid + (e >> 1) * 8;
-                float sv = key >= nlo && key < n ? s[i][e] * a.scale : -INFINITY;
+                float sv = key >= nlo && key < n ? capped(a, s[i][e] * a.scale) : -INFINITY;
                 // (with a distance bias the tiles come by copies, so jt + key is the position)
                 if (!TMA && a.dist_bias && row < gc && key >= nlo && key < n)
                     sv += distance_bias(a, p, jt + key, h0 + row);
@@ -966,7 +986,7 @@ attention_decode_mma_kernel(DecodeArgs a, int cs, FuseQK fq,
             const int key = warp * 8 + tig * 2 + (e & 1);
             const int row = gid + (e >> 1) * 8;
             float sv = key >= nlo && key < n
-                ? ((s[0][e] + s[1][e]) + (s[2][e] + s[3][e])) * a.scale : -INFINITY;
+                ? capped(a, ((s[0][e] + s[1][e]) + (s[2][e] + s[3][e])) * a.scale) : -INFINITY;
             if (!TMA && a.dist_bias && row < gc && key >= nlo && key < n)
                 sv += distance_bias(a, p, jt + key, h0 + row);
             Ss[row * DM_KEYS + key] = sv;
@@ -1047,7 +1067,7 @@ attention_decode_mma_kernel(DecodeArgs a, int cs, FuseQK fq,
 #pragma unroll
         for (int i = 0; i < NP * 2; ++i) {
             const int d = warp * Sh::DW + i * 8 + tig * 2;
-            if (d >= hd) continue;
+            if (d >= hdv) continue;
 #pragma unroll
             for (int half = 0; half < 2; ++half) {
                 const int row = gid + half * 8;
@@ -1055,14 +1075,14 @@ attention_decode_mma_kernel(DecodeArgs a, int cs, FuseQK fq,
                 const float v0 = o[i][half * 2], v1 = o[i][half * 2 + 1];
                 if (used == 1) {
                     const float inv = 1.0f / (stat[row * 2 + 1] + sink_term(a, h0 + row, stat[row * 2]));
-                    outp[row * hd + d] = __float2bfloat16_rn(v0 * inv);
-                    outp[row * hd + d + 1] = __float2bfloat16_rn(v1 * inv);
+                    outp[row * hdv + d] = __float2bfloat16_rn(v0 * inv);
+                    outp[row * hdv + d + 1] = __float2bfloat16_rn(v1 * inv);
                 } else if (cs > 1) {
                     Osm[row * HDP + d] = v0;
                     Osm[row * HDP + d + 1] = v1;
                 } else {
                     float* dst = a.part_acc +
-                                 (((size_t)b * a.nh + h0 + row) * a.n_splits + split) * hd + d;
+                                 (((size_t)b * a.nh + h0 + row) * a.n_splits + split) * hdv + d;
                     dst[0] = v0;
                     dst[1] = v1;
                 }
@@ -1108,11 +1128,11 @@ attention_decode_mma_kernel(DecodeArgs a, int cs, FuseQK fq,
                     O = fmaf(w, oq[q], O);
                 }
             }
-            if (d < hd) {
+            if (d < hdv) {
                 if (used_clusters == 1) {
-                    outp[row * hd + d] = __float2bfloat16_rn(O / (L + sink_term(a, h0 + row, M)));
+                    outp[row * hdv + d] = __float2bfloat16_rn(O / (L + sink_term(a, h0 + row, M)));
                 } else {
-                    a.part_acc[(((size_t)b * a.nh + h0 + row) * a.n_splits + cid) * hd + d] = O;
+                    a.part_acc[(((size_t)b * a.nh + h0 + row) * a.n_splits + cid) * hdv + d] = O;
                     if (d == 0) {
                         float* ml = a.part_ml + (((size_t)b * a.nh + h0 + row) * a.n_splits + cid) * 2;
                         ml[0] = M;
@@ -1250,7 +1270,7 @@ int launch_decode_mma(const DecodeArgs& a0, int B, cudaStream_t stream, const Fu
 // tiles' (pages of 64 positions, a ring of whole pages, a head as wide as its tile).
 template <int HDP>
 int launch_decode_form(const DecodeArgs& a, int B, cudaStream_t stream, const FuseQK& fq) {
-    const bool can = a.page == DM_KEYS && a.cap % DM_KEYS == 0 && a.hd == HDP &&
+    const bool can = a.page == DM_KEYS && a.cap % DM_KEYS == 0 && a.hd == HDP && a.hdv == HDP &&
                      agv_aligned(a.k_pool, 128) && agv_aligned(a.v_pool, 128);
     const int form = decode_tiles_form();
     // A request by TMA saves its time per tile, and a window that does not start on a page
@@ -1280,14 +1300,14 @@ int launch_decode_form(const DecodeArgs& a, int B, cudaStream_t stream, const Fu
     return launch_decode_mma<HDP, false>(a, B, stream, fq);
 }
 
-int pick_chunk(int hd, int elem) {
+int pick_chunk(int hd, int elem) {                  // hd: the wider of a key and a value head
     int ch = 64;
     while (ch > 8 && (size_t)2 * ch * hd * elem > 128 * 1024) ch /= 2;
     return ch;
 }
 
-size_t split_smem(int hd, int ch, int elem) {
-    return (size_t)2 * ch * hd * elem + (size_t)AD_GC * hd * 4 + (size_t)AD_GC * ch * 4 +
+size_t split_smem(int hd, int hdv, int ch, int elem) {
+    return (size_t)ch * (hd + hdv) * elem + (size_t)AD_GC * hd * 4 + (size_t)AD_GC * ch * 4 +
            AD_GC * 2 * 4 + (size_t)ch * 4;
 }
 
@@ -1321,7 +1341,13 @@ static int attention_decode_impl(const void* q, long long q_stride, void* out, i
                                  int max_keys, float* part_acc, float* part_ml, int* counters,
                                  cudaStream_t stream, const FuseQK& fq,
                                  const float* sinks = nullptr, const float* dist_bias = nullptr,
-                                 int n_dist = 0, int keep_first = 0) {
+                                 int n_dist = 0, int keep_first = 0, int hdv = 0,
+                                 float softcap = 0.f) {
+    if (hdv == 0) hdv = hd;
+    AGV_REQUIRE(hdv == hd || (hdv > 0 && hdv % 16 == 0 && hdv <= AD_MAX_HD && !fq.part),
+                "attention_decode: value heads of %d must be a multiple of 16 up to %d, with "
+                "finished queries", hdv, AD_MAX_HD);
+    const int wide = hd > hdv ? hd : hdv;
     AGV_REQUIRE(B >= 0 && nh > 0 && nkv > 0 && hd > 0, "attention_decode: bad sizes");
     AGV_REQUIRE(keep_first >= 0 && (keep_first == 0 || (window > 0 && !dist_bias && !fq.part)),
                 "attention_decode: kept first keys go with a sliding window, without a distance "
@@ -1346,18 +1372,18 @@ static int attention_decode_impl(const void* q, long long q_stride, void* out, i
     AGV_REQUIRE(B <= 65535, "attention_decode: batch %d exceeds the grid limit", B);
     AGV_REQUIRE(part_acc && part_ml && counters, "attention_decode: scratch pointers are null");
     if (B == 0) return 0;
-    const int ch = pick_chunk(hd, elem);
+    const int ch = pick_chunk(wide, elem);
     const int n_splits = (max_keys + ch - 1) / ch;
-    const size_t smem = split_smem(hd, ch, elem);
+    const size_t smem = split_smem(hd, hdv, ch, elem);
     AGV_REQUIRE(smem <= (size_t)AD_MAX_SMEM, "attention_decode: %zu bytes of shared memory needed",
                 smem);
     DecodeArgs a{q, q_stride, out, k_pool, v_pool, page_table, slots, positions, part_acc, part_ml,
                  counters, max_pages, page, cap, nh, nkv, hd, window, n_splits, ch, scale, sinks,
-                 dist_bias, n_dist, keep_first};
-    if (dtype == AGV_BF16 && hd % 8 == 0 && hd <= 256 && ch == DM_KEYS &&
+                 dist_bias, n_dist, keep_first, softcap, hdv};
+    if (dtype == AGV_BF16 && hd % 8 == 0 && wide <= 256 && ch == DM_KEYS &&
         (fq.part || (q_stride % 8 == 0 && agv_aligned(q, 16)))) {
-        if (hd <= 64) return launch_decode_form<64>(a, B, stream, fq);
-        if (hd <= 128) return launch_decode_form<128>(a, B, stream, fq);
+        if (wide <= 64) return launch_decode_form<64>(a, B, stream, fq);
+        if (wide <= 128) return launch_decode_form<128>(a, B, stream, fq);
         return launch_decode_form<256>(a, B, stream, fq);
     }
     AGV_REQUIRE(!fq.part, "attention_decode: the fused form needs the tensor-core kernel");
@@ -1427,17 +1453,19 @@ AGV_API int agv_attention_decode_ex2(const void* q, long long q_stride, void* ou
 // The same with kept first keys: position p also sees the keys j < keep_first behind its
 // window.  max_keys then counts them: at least position - window start + 1 + min(keep_first,
 // window start) of every entry.  The cache entry must keep every key (cap above every position).
+// hdv: the value head size (out [B, nh * hdv]; the plan and the scratch are those of the wider
+// of hd and hdv); 0: hd.  softcap > 0: the scaled score s becomes softcap * tanh(s / softcap).
 AGV_API int agv_attention_decode_ex3(const void* q, long long q_stride, void* out, int dtype,
                                      const void* k_pool, const void* v_pool, const int* page_table,
                                      const int* slots, const int* positions, int max_pages, int page,
                                      int cap, int B, int nh, int nkv, int hd, float scale, int window,
                                      int max_keys, float* part_acc, float* part_ml, int* counters,
                                      const float* sinks, const float* dist_bias, int n_dist,
-                                     int keep_first, cudaStream_t stream) {
+                                     int keep_first, int hdv, float softcap, cudaStream_t stream) {
     return attention_decode_impl(q, q_stride, out, dtype, k_pool, v_pool, page_table, slots,
                                  positions, max_pages, page, cap, B, nh, nkv, hd, scale, window,
                                  max_keys, part_acc, part_ml, counters, stream, FuseQK{}, sinks,
-                                 dist_bias, n_dist, keep_first);
+                                 dist_bias, n_dist, keep_first, hdv, softcap);
 }
 
 // Whether agv_attention_decode_fused takes these sizes: bfloat16, head sizes 64, 128,

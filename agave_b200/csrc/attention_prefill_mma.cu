@@ -85,7 +85,8 @@ attention_prefill_mma_kernel(const __nv_bfloat16* __restrict__ q, long long q_st
                              __nv_bfloat16* __restrict__ out, const int* __restrict__ cu_seqlens,
                              int nh, int nkv, int hd, float scale_log2e, int window,
                              const float* __restrict__ sinks, int hdv, long long v_stride,
-                             const float* __restrict__ dist_bias, int n_dist, int keep_first) {
+                             const float* __restrict__ dist_bias, int n_dist, int keep_first,
+                             float softcap) {
     pdl_wait();
     pdl_launch_next();
     constexpr int FA_M = NW * 16, FA_THREADS = NW * 32;
@@ -128,6 +129,7 @@ attention_prefill_mma_kernel(const __nv_bfloat16* __restrict__ q, long long q_st
     for (int i = 0; i < HDP / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
     float row_m[2] = {-INFINITY, -INFINITY}, row_l[2] = {0.f, 0.f};
     const int qrow = m0 + warp * 16 + gid;             // this thread's rows: qrow, qrow + 8
+    const float cap_in = 2.0f * 1.4426950408889634f / softcap;
 
     for (int it = 0; it < n_walk; ++it) {
         const int t = tile_of(it);
@@ -169,6 +171,8 @@ attention_prefill_mma_kernel(const __nv_bfloat16* __restrict__ q, long long q_st
                 float val = -INFINITY;
                 if (ok) {
                     val = s[i][e] * scale_log2e;
+                    // (scale and cap carry log2(e): the capped score is on the same scale)
+                    if (softcap > 0.f) val = soft_capped_ex2(val, cap_in, softcap);
                     // a learned bias by distance, on the same base-2 scale as the score
                     if (dist_bias)
                         val += dist_bias[(size_t)h * n_dist + min(p - j, n_dist - 1)] * 1.4426950408889634f;
@@ -256,7 +260,8 @@ template <int HDP, int NW>
 int launch_fa(const void* q, long long q_stride, const void* k, const void* v, long long kv_stride,
               void* out, const int* cu_seqlens, int B, int max_len, int nh, int nkv, int hd,
               float scale, int window, cudaStream_t stream, const float* sinks, int hdv,
-              long long v_stride, const float* dist_bias, int n_dist, int keep_first) {
+              long long v_stride, const float* dist_bias, int n_dist, int keep_first,
+              float softcap) {
     auto kern = attention_prefill_mma_kernel<HDP, NW>;
     constexpr int FA_M = NW * 16, FA_THREADS = NW * 32;
     constexpr int smem = (FA_M + 2 * FA_N) * HDP * 2;
@@ -268,7 +273,8 @@ int launch_fa(const void* q, long long q_stride, const void* k, const void* v, l
     dim3 grid((max_len + FA_M - 1) / FA_M, nh, B);
     agv_launch(kern, grid, FA_THREADS, smem, stream, (const __nv_bfloat16*)q, q_stride, (const __nv_bfloat16*)k, (const __nv_bfloat16*)v,
         kv_stride, (__nv_bfloat16*)out, cu_seqlens, nh, nkv, hd,
-        scale * 1.4426950408889634f, window, sinks, hdv, v_stride, dist_bias, n_dist, keep_first);
+        scale * 1.4426950408889634f, window, sinks, hdv, v_stride, dist_bias, n_dist, keep_first,
+        softcap * 1.4426950408889634f);
     AGV_LAUNCH_OK("attention_prefill_mma_kernel");
     return 0;
 }
@@ -294,7 +300,8 @@ AGV_API int agv_attention_prefill_mma_ex3(const void* q, long long q_stride, con
                                           const int* cu_seqlens, int B, int max_len, int nh, int nkv,
                                           int hd, float scale, int window, const float* sinks,
                                           int hdv, long long v_stride, const float* dist_bias,
-                                          int n_dist, int keep_first, cudaStream_t stream);
+                                          int n_dist, int keep_first, float softcap,
+                                          cudaStream_t stream);
 
 AGV_API int agv_attention_prefill_mma_ex2(const void* q, long long q_stride, const void* k,
                                           const void* v, long long kv_stride, void* out,
@@ -304,16 +311,18 @@ AGV_API int agv_attention_prefill_mma_ex2(const void* q, long long q_stride, con
                                           int n_dist, cudaStream_t stream) {
     return agv_attention_prefill_mma_ex3(q, q_stride, k, v, kv_stride, out, cu_seqlens, B, max_len,
                                          nh, nkv, hd, scale, window, sinks, hdv, v_stride,
-                                         dist_bias, n_dist, 0, stream);
+                                         dist_bias, n_dist, 0, 0.f, stream);
 }
 
-// keep_first: with a sliding window, position p also sees the keys j < keep_first.
+// keep_first: with a sliding window, position p also sees the keys j < keep_first.  softcap >
+// 0: the scaled score s becomes softcap * tanh(s / softcap), before a distance bias.
 AGV_API int agv_attention_prefill_mma_ex3(const void* q, long long q_stride, const void* k,
                                           const void* v, long long kv_stride, void* out,
                                           const int* cu_seqlens, int B, int max_len, int nh, int nkv,
                                           int hd, float scale, int window, const float* sinks,
                                           int hdv, long long v_stride, const float* dist_bias,
-                                          int n_dist, int keep_first, cudaStream_t stream) {
+                                          int n_dist, int keep_first, float softcap,
+                                          cudaStream_t stream) {
     AGV_REQUIRE(keep_first >= 0 && (keep_first == 0 || window > 0),
                 "attention: kept first keys go with a sliding window");
     AGV_REQUIRE(B >= 0 && nh > 0 && nkv > 0 && hd > 0 && max_len >= 0, "attention: bad sizes");
@@ -334,10 +343,10 @@ AGV_API int agv_attention_prefill_mma_ex3(const void* q, long long q_stride, con
 #define AGV_FA(HDP)                                                                             \
     return wide ? launch_fa<HDP, 8>(q, q_stride, k, v, kv_stride, out, cu_seqlens, B, max_len,  \
                                     nh, nkv, hd, scale, window, stream, sinks, hdv, v_stride,    \
-                                    dist_bias, n_dist, keep_first)                               \
+                                    dist_bias, n_dist, keep_first, softcap)                             \
                 : launch_fa<HDP, 4>(q, q_stride, k, v, kv_stride, out, cu_seqlens, B, max_len,  \
                                     nh, nkv, hd, scale, window, stream, sinks, hdv, v_stride,    \
-                                    dist_bias, n_dist, keep_first)
+                                    dist_bias, n_dist, keep_first, softcap)
     const int widest = hd > hdv ? hd : hdv;
     if (widest <= 64) AGV_FA(64);
     if (widest <= 128) AGV_FA(128);

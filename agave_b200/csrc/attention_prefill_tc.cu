@@ -50,9 +50,10 @@ constexpr float AT_LAZY = 8.0f;    // log2 units the maximum may lag before O is
 __device__ int g_attn_status = 0;  // 0 ok; else (role << 8) | detail of the first wait that gave up
 
 struct AtArgs {
-    __nv_bfloat16* out;            // [T, nh * hd]
+    __nv_bfloat16* out;            // [T, nh * hdv]
     const int* cu;                 // [B + 1]
     int nh, nkv, hd, G, QT;        // G heads packed per CTA, QT = 128 / G tokens
+    int hdv;                       // the value head size (out is [T, nh * hdv])
     int window;
     int keep_first;                // with a window: the first keys that stay visible behind it
     float scale_log2e;
@@ -62,6 +63,9 @@ struct AtArgs {
     const float* dist_bias;        // [nh, n_dist] learned bias by distance (unscaled), or null
     int n_dist;
     float inv_scale;               // 1 / scale: the bias joins the raw scores before the scale
+    // the soft cap (CAP): a raw score z becomes cap * tanh(z * scale / cap); scale_log2e is then
+    // log2(e) alone
+    float cap, cap_in;             // cap_in = 2 log2(e) * scale / cap
 };
 
 // 2^x by the hardware approximation (relative error about 2^-22; -inf gives 0).
@@ -113,9 +117,9 @@ transpose_values_kernel(const __nv_bfloat16* __restrict__ v, long long kv_stride
 }
 
 // ------------------------------------------------------------------ attention
-// BIAS: the form that adds a table value to every score (a form of its own, so that the plain
-// form's softmax loop keeps its registers)
-template <bool BIAS>
+// BIAS: the form that adds a table value to every score; CAP: the form with a soft cap on the
+// scores (forms of their own, so that the plain form's softmax loop keeps its registers)
+template <bool BIAS, bool CAP>
 __global__ void __launch_bounds__(AT_THREADS, 1)
 attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
                             const __grid_constant__ CUtensorMap map_k,
@@ -128,7 +132,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
     uint8_t* smem = (uint8_t*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
     const int q_bytes = a.kb * AT_M * 128;              // [kb][128 rows][128 B]
     const int k_bytes = a.kb * AT_N * 128;              // [kb][64 keys][128 B]
-    const int v_bytes = a.hd * 128;                     // [hd rows][64 keys]
+    const int v_bytes = a.hdv * 128;                    // [hdv rows][64 keys]
     constexpr int p_bytes = AT_M * 128;                 // [128 rows][64 keys]
     uint8_t* Qs = smem;
     uint8_t* Ks = Qs + q_bytes;                         // two stages
@@ -231,7 +235,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
                 return false;
             }
             mbar_expect_tx(&v_full[s], (uint32_t)v_bytes);
-            tma_load_2d(Vs + s * v_stage, &map_vt, vt0 + tile_of(j) * AT_N, kvh * a.hd, &v_full[s]);
+            tma_load_2d(Vs + s * v_stage, &map_vt, vt0 + tile_of(j) * AT_N, kvh * a.hdv, &v_full[s]);
             return true;
         };
         // keys run one tile ahead of values: K of tile j + 1 is wanted before V of tile j
@@ -291,7 +295,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
         }
     } else if (warp == 6 && lane == 0) {
         // ------------------------------------------------------------ O += P V
-        const uint32_t idesc_o = umma_idesc(AT_M, a.hd);
+        const uint32_t idesc_o = umma_idesc(AT_M, a.hdv);
         const uint64_t v_desc0 = umma_desc(smem_u32(Vs)), p_desc0 = umma_desc(smem_u32(Ps));
         for (int i = 0; i < n_tiles && !*abort_flag; ++i) {
             const int s = i & 1;
@@ -340,6 +344,15 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
             tc_fence_before();
             __syncwarp();
             if (lane == 0) mbar_arrive(&s_free[s]);
+            if (CAP) {
+                // (before the bounds: a capped -infinity is -cap)
+#pragma unroll
+                for (int c = 0; c < 64; ++c) {
+                    const float e = ex2_fast(__uint_as_float(sr[c >> 4][c & 15]) * a.cap_in);
+                    sr[c >> 4][c & 15] =
+                        __float_as_uint(fmaf(__fdividef(2.0f, 1.0f + e), -a.cap, a.cap));
+                }
+            }
             const int j0 = tile_of(j) * AT_N;
             // a tile every row of the CTA sees whole needs no bounds
             const bool whole = j0 + AT_N - 1 <= q_min &&
@@ -421,7 +434,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
                 }
                 tc_fence_after();
                 if (__any_sync(0xffffffffu, rescale)) {
-                    for (int c = 0; c < a.hd; c += 16) {
+                    for (int c = 0; c < a.hdv; c += 16) {
                         uint32_t o[16];
                         tc_ld16(lane_addr + AT_O_COL + c, o);
                         tc_wait_ld();
@@ -450,21 +463,21 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
                 if (a.sinks && m_used != -INFINITY)
                     l += exp2f(a.sinks[head0 + hl] * 1.4426950408889634f - m_used);
                 const float inv = l > 0.f ? 1.0f / l : 0.f;
-                __nv_bfloat16* dst = a.out + (size_t)(seq0 + qp) * ((size_t)a.nh * a.hd) +
-                                     (size_t)(head0 + hl) * a.hd;
+                __nv_bfloat16* dst = a.out + (size_t)(seq0 + qp) * ((size_t)a.nh * a.hdv) +
+                                     (size_t)(head0 + hl) * a.hdv;
                 const bool valid = qp < len;
                 // 64 columns per wait: four loads in flight, then their stores
-                for (int c0 = 0; c0 < a.hd; c0 += 64) {
+                for (int c0 = 0; c0 < a.hdv; c0 += 64) {
                     uint32_t o[4][16];
 #pragma unroll
                     for (int q = 0; q < 4; ++q)
-                        if (c0 + q * 16 < a.hd) tc_ld16(lane_addr + AT_O_COL + c0 + q * 16, o[q]);
+                        if (c0 + q * 16 < a.hdv) tc_ld16(lane_addr + AT_O_COL + c0 + q * 16, o[q]);
                     tc_wait_ld();
                     if (valid) {
 #pragma unroll
                         for (int q = 0; q < 4; ++q) {
                             const int c = c0 + q * 16;
-                            if (c < a.hd) {
+                            if (c < a.hdv) {
                                 uint32_t w[8];
 #pragma unroll
                                 for (int i = 0; i < 8; ++i) {
@@ -589,7 +602,8 @@ AGV_API int agv_attention_prefill_tc_ex3(const void* q, long long q_stride, cons
                                          long long vt_cols, int vt_ready, const int* cu_seqlens, int B,
                                          int T, int max_len, int nh, int nkv, int hd, float scale,
                                          int window, const float* sinks, const float* dist_bias,
-                                         int n_dist, int keep_first, cudaStream_t stream);
+                                         int n_dist, int keep_first, int hdv, long long v_stride,
+                                         float softcap, cudaStream_t stream);
 
 AGV_API int agv_attention_prefill_tc_ex(const void* q, long long q_stride, const void* k,
                                         const void* v, long long kv_stride, void* out, void* vt,
@@ -611,17 +625,20 @@ AGV_API int agv_attention_prefill_tc_ex2(const void* q, long long q_stride, cons
                                          int n_dist, cudaStream_t stream) {
     return agv_attention_prefill_tc_ex3(q, q_stride, k, v, kv_stride, out, vt, vt_cols, vt_ready,
                                         cu_seqlens, B, T, max_len, nh, nkv, hd, scale, window, sinks,
-                                        dist_bias, n_dist, 0, stream);
+                                        dist_bias, n_dist, 0, hd, kv_stride, 0.f, stream);
 }
 
 // The same with kept first keys: with a sliding window, position p also sees the keys
-// j < keep_first.
+// j < keep_first.  hdv, v_stride: the value head size (a multiple of 16 up to 256) and the value
+// rows' stride (out is [T, nh * hdv] and vt [nkv * hdv, vt_cols]).  softcap > 0: the scaled score
+// s becomes softcap * tanh(s / softcap); not with a distance bias.
 AGV_API int agv_attention_prefill_tc_ex3(const void* q, long long q_stride, const void* k,
                                          const void* v, long long kv_stride, void* out, void* vt,
                                          long long vt_cols, int vt_ready, const int* cu_seqlens, int B,
                                          int T, int max_len, int nh, int nkv, int hd, float scale,
                                          int window, const float* sinks, const float* dist_bias,
-                                         int n_dist, int keep_first, cudaStream_t stream) {
+                                         int n_dist, int keep_first, int hdv, long long v_stride,
+                                         float softcap, cudaStream_t stream) {
     AGV_REQUIRE(scale > 0.f, "attention: the tcgen05 kernel takes a positive score scale");
     AGV_REQUIRE(keep_first >= 0 && (keep_first == 0 || window > 0),
                 "attention: kept first keys go with a sliding window");
@@ -639,19 +656,25 @@ AGV_API int agv_attention_prefill_tc_ex3(const void* q, long long q_stride, cons
                 "attention: the transposed-values scratch has %lld columns, %lld are needed",
                 vt_cols, agv_attention_prefill_tc_vt_cols(T, B));
     AGV_REQUIRE(B <= 65535 && nh <= 65535, "attention: batch or head count exceeds the grid limit");
+    AGV_REQUIRE(hdv > 0 && hdv % 16 == 0 && hdv <= 256 && v_stride % 8 == 0,
+                "attention: the value head size (%d) must be a multiple of 16 up to 256", hdv);
+    AGV_REQUIRE(softcap <= 0.f || !dist_bias, "attention: a soft cap goes without a distance bias");
     if (B == 0 || max_len == 0 || T == 0) return 0;
 
     AtArgs a;
     a.out = (__nv_bfloat16*)out;
     a.cu = cu_seqlens;
-    a.nh = nh, a.nkv = nkv, a.hd = hd;
+    a.nh = nh, a.nkv = nkv, a.hd = hd, a.hdv = hdv;
     a.G = packed_heads(nh, nkv);
     a.QT = AT_M / a.G;
     a.window = window;
     a.keep_first = keep_first;
-    a.scale_log2e = scale * 1.4426950408889634f;
+    const bool cap = softcap > 0.f;
+    a.scale_log2e = (cap ? 1.0f : scale) * 1.4426950408889634f;
+    a.cap = softcap;
+    a.cap_in = cap ? 2.0f * 1.4426950408889634f * scale / softcap : 0.f;
     a.kb = (hd + 63) / 64;
-    a.tmem_cols = AT_O_COL + hd <= 256 ? 256 : 512;
+    a.tmem_cols = AT_O_COL + hdv <= 256 ? 256 : 512;
     a.sinks = sinks;
     a.dist_bias = dist_bias;
     a.n_dist = n_dist;
@@ -671,35 +694,31 @@ AGV_API int agv_attention_prefill_tc_ex3(const void* q, long long q_stride, cons
         if (int rc = make_map_nd(&mk, k, 3, dims, str, box)) return rc;
     }
     {
-        cuuint64_t dims[2] = {(cuuint64_t)vt_cols, (cuuint64_t)nkv * hd};
+        cuuint64_t dims[2] = {(cuuint64_t)vt_cols, (cuuint64_t)nkv * hdv};
         cuuint64_t str[1] = {(cuuint64_t)vt_cols * 2};
-        cuuint32_t box[2] = {64, (cuuint32_t)hd};
+        cuuint32_t box[2] = {64, (cuuint32_t)hdv};
         if (int rc = make_map_nd(&mvt, vt, 2, dims, str, box)) return rc;
     }
 
     if (!vt_ready)
-        if (int rc = agv_transpose_values(v, kv_stride, vt, vt_cols, cu_seqlens, B, max_len, nkv, hd,
+        if (int rc = agv_transpose_values(v, v_stride, vt, vt_cols, cu_seqlens, B, max_len, nkv, hdv,
                                           stream))
             return rc;
-    const int v_stage = (hd * 128 + 1023) & ~1023;
+    const int v_stage = (hdv * 128 + 1023) & ~1023;
     const size_t smem = 1024 + (size_t)a.kb * AT_M * 128 + 2 * (size_t)a.kb * AT_N * 128 +
                         2 * (size_t)v_stage + 2 * (size_t)AT_M * 128 + 256;
-    static size_t configured[2] = {0, 0};
-    const int form = dist_bias ? 1 : 0;
+    static size_t configured[3] = {0, 0, 0};
+    const int form = dist_bias ? 1 : cap ? 2 : 0;
+    auto kern = form == 1   ? attention_prefill_tc_kernel<true, false>
+                : form == 2 ? attention_prefill_tc_kernel<false, true>
+                            : attention_prefill_tc_kernel<false, false>;
     if (smem > configured[form]) {
-        if (form)
-            AGV_CUDA_OK(cudaFuncSetAttribute(attention_prefill_tc_kernel<true>,
-                                             cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-        else
-            AGV_CUDA_OK(cudaFuncSetAttribute(attention_prefill_tc_kernel<false>,
-                                             cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+        AGV_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                         (int)smem));
         configured[form] = smem;
     }
     dim3 grid((max_len + a.QT - 1) / a.QT, a.G > 1 ? nkv : nh, B);
-    if (form)
-        agv_launch(attention_prefill_tc_kernel<true>, grid, AT_THREADS, smem, stream, mq, mk, mvt, a);
-    else
-        agv_launch(attention_prefill_tc_kernel<false>, grid, AT_THREADS, smem, stream, mq, mk, mvt, a);
+    agv_launch(kern, grid, AT_THREADS, smem, stream, mq, mk, mvt, a);
     AGV_LAUNCH_OK("attention_prefill_tc_kernel");
     return 0;
 }

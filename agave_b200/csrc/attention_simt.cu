@@ -17,6 +17,7 @@
 // With a sliding window, the sequence's first keep_first keys may stay visible behind it.
 // A bias per (distance, head) may be added to the scaled score, and the cache's value rows
 // may lie at a stride of their own (values that are the leading part of the key rows).
+// A soft cap may turn the scaled score s into cap * tanh(s / cap) (before a bias by distance).
 #include "common.cuh"
 
 constexpr int AT_WARPS = 4;
@@ -44,7 +45,8 @@ attention_simt_kernel(const T* __restrict__ q, long long q_stride, const T* __re
                       const int* __restrict__ positions, const int* __restrict__ seq_index,
                       const int* __restrict__ cu_seqlens, PagedKV pk, int n_tokens, int nh, int nkv,
                       int hd, float scale, int window, int hdv, long long v_stride,
-                      const float* __restrict__ sinks, DistanceBias db, int keep_first) {
+                      const float* __restrict__ sinks, DistanceBias db, int keep_first,
+                      float softcap) {
     pdl_wait();
     pdl_launch_next();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -96,6 +98,7 @@ attention_simt_kernel(const T* __restrict__ q, long long q_stride, const T* __re
             if (e < hd) s = fmaf(qr[i], to_f32(kp[e]), s);
         }
         s = warp_sum(s) * scale;
+        if (softcap > 0.f) s = soft_capped(s, softcap);
         if (db.bias) s += db.bias[(size_t)h * db.n + min(p - j, db.n - 1)];
         const float mn = fmaxf(m, s);
         const float alpha = expf(m - mn);      // exp(-inf) = 0 on the first key
@@ -148,7 +151,7 @@ AGV_API int agv_attention_prefill_simt_ex(const void* q, long long q_stride, con
                                           int hd, float scale, int window, int hdv,
                                           long long v_stride, const float* sinks,
                                           const float* dist_bias, int n_dist, int keep_first,
-                                          cudaStream_t stream) {
+                                          float softcap, cudaStream_t stream) {
     if (int rc = check_attn(n_tokens, nh, nkv, hd, window, hdv)) return rc;
     AGV_REQUIRE(!dist_bias || n_dist > 0, "attention: an empty distance table");
     if (n_tokens == 0) return 0;
@@ -159,11 +162,11 @@ AGV_API int agv_attention_prefill_simt_ex(const void* q, long long q_stride, con
     if (dtype == AGV_F32)
         agv_launch(attention_simt_kernel<float, false>, grid, AT_WARPS * 32, 0, stream, (const float*)q, q_stride, (const float*)k, (const float*)v, kv_stride, (float*)out,
             positions, seq_index, cu_seqlens, pk, n_tokens, nh, nkv, hd, scale, window, hdv,
-            v_stride, sinks, db, keep_first);
+            v_stride, sinks, db, keep_first, softcap);
     else if (dtype == AGV_BF16)
         agv_launch(attention_simt_kernel<__nv_bfloat16, false>, grid, AT_WARPS * 32, 0, stream, (const __nv_bfloat16*)q, q_stride, (const __nv_bfloat16*)k, (const __nv_bfloat16*)v,
             kv_stride, (__nv_bfloat16*)out, positions, seq_index, cu_seqlens, pk, n_tokens, nh,
-            nkv, hd, scale, window, hdv, v_stride, sinks, db, keep_first);
+            nkv, hd, scale, window, hdv, v_stride, sinks, db, keep_first, softcap);
     else
         return agv_fail(-1, "attention: unknown dtype %d", dtype);
     AGV_LAUNCH_OK("attention_simt_kernel");
@@ -177,7 +180,7 @@ AGV_API int agv_attention_prefill_simt(const void* q, long long q_stride, const 
                                        float scale, int window, cudaStream_t stream) {
     return agv_attention_prefill_simt_ex(q, q_stride, k, v, kv_stride, out, dtype, positions,
                                          seq_index, cu_seqlens, n_tokens, nh, nkv, hd, scale,
-                                         window, hd, kv_stride, nullptr, nullptr, 0, 0, stream);
+                                         window, hd, kv_stride, nullptr, nullptr, 0, 0, 0.f, stream);
 }
 
 // Queries against the paged cache (the query's own key is already stored).
@@ -191,7 +194,7 @@ AGV_API int agv_attention_paged_simt_ex(const void* q, long long q_stride, void*
                                         int page, int cap, int n_tokens, int nh, int nkv, int hd,
                                         float scale, int window, int hdv, const float* sinks,
                                         const float* dist_bias, int n_dist, int v_row, int keep_first,
-                                        cudaStream_t stream) {
+                                        float softcap, cudaStream_t stream) {
     if (int rc = check_attn(n_tokens, nh, nkv, hd, window, hdv)) return rc;
     AGV_REQUIRE(!dist_bias || n_dist > 0, "attention: an empty distance table");
     AGV_REQUIRE(v_row == 0 || v_row >= nkv * hdv, "attention: value rows overlap");
@@ -207,10 +210,10 @@ AGV_API int agv_attention_paged_simt_ex(const void* q, long long q_stride, void*
     PagedKV pk{k_pool, v_pool, page_table, slots, max_pages, page, cap, v_row ? v_row : nkv * hdv};
     if (dtype == AGV_F32)
         agv_launch(attention_simt_kernel<float, true>, grid, AT_WARPS * 32, 0, stream, (const float*)q, q_stride, nullptr, nullptr, 0, (float*)out, positions, seq_index,
-            nullptr, pk, n_tokens, nh, nkv, hd, scale, window, hdv, 0LL, sinks, db, keep_first);
+            nullptr, pk, n_tokens, nh, nkv, hd, scale, window, hdv, 0LL, sinks, db, keep_first, softcap);
     else if (dtype == AGV_BF16)
         agv_launch(attention_simt_kernel<__nv_bfloat16, true>, grid, AT_WARPS * 32, 0, stream, (const __nv_bfloat16*)q, q_stride, nullptr, nullptr, 0, (__nv_bfloat16*)out, positions,
-            seq_index, nullptr, pk, n_tokens, nh, nkv, hd, scale, window, hdv, 0LL, sinks, db, keep_first);
+            seq_index, nullptr, pk, n_tokens, nh, nkv, hd, scale, window, hdv, 0LL, sinks, db, keep_first, softcap);
     else
         return agv_fail(-1, "attention: unknown dtype %d", dtype);
     AGV_LAUNCH_OK("attention_simt_kernel");
@@ -225,5 +228,5 @@ AGV_API int agv_attention_paged_simt(const void* q, long long q_stride, void* ou
                                      cudaStream_t stream) {
     return agv_attention_paged_simt_ex(q, q_stride, out, dtype, k_pool, v_pool, page_table, slots,
                                        positions, seq_index, max_pages, page, cap, n_tokens, nh,
-                                       nkv, hd, scale, window, hd, nullptr, nullptr, 0, 0, 0, stream);
+                                       nkv, hd, scale, window, hd, nullptr, nullptr, 0, 0, 0, 0.f, stream);
 }

@@ -121,6 +121,16 @@ __host__ __device__ __forceinline__ int first_visible(int p, int window) {
     return 0;
 }
 
+// An attention score under a soft cap: cap * tanh(score / cap).  The second form takes
+// 2 log2(e) / cap and goes by tanh(x) = 1 - 2 / (1 + e^2x), whose absolute error is a few
+// roundings of cap (-inf gives -cap: masks are applied after the cap).
+__device__ __forceinline__ float soft_capped(float score, float cap) {
+    return cap * tanhf(score / cap);
+}
+__device__ __forceinline__ float soft_capped_ex2(float score, float two_log2e_over_cap, float cap) {
+    return fmaf(__fdividef(2.0f, 1.0f + exp2f(score * two_log2e_over_cap)), -cap, cap);
+}
+
 __device__ __forceinline__ float to_f32(float v) { return v; }
 __device__ __forceinline__ float to_f32(__nv_bfloat16 v) { return __bfloat162float(v); }
 template <typename T> __device__ __forceinline__ T from_f32(float v);

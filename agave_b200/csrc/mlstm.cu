@@ -19,6 +19,9 @@
 //    token are read by a whole warp at once; the row blocks' parts of a column's dot product
 //    with q meet in shared memory after a chunk of tokens.  It leaves S_t^T q_t, n_t . q_t
 //    and exp(-m_t).
+//  * agv_head_scan: the same kernel without n and m, for other recurrences S_t = a_t S_(t-1) +
+//    b_t k_t v_t^T, o_t = S_t^T q_t with a pair (a_t, b_t) per head and token that is given; the
+//    heads of a group may share q and k (the state-space form of Mamba-2).
 //  * agv_mlstm_out: the division, every head's o over its root mean square, times a weight
 //    per channel, times sigmoid(g), rounded to the compute dtype for the output product.
 #include "common.cuh"
@@ -87,11 +90,19 @@ template <int N> __device__ __forceinline__ void cp_async_wait() {
 // kernel's.  Every group of eight columns has a copy of the head's running maximum in the
 // state; a CTA reads its first group's and writes all of its groups', so that no CTA reads
 // what another writes.
-template <int RW>
-__global__ void __launch_bounds__((RW + 1) * 32)
-mlstm_scan_kernel(const float* __restrict__ qkv, const float* __restrict__ gates,
-                  float* __restrict__ num, float* __restrict__ den, int H, int d, int dv,
-                  float* __restrict__ state, long long state_stride,
+//
+// NORM false: there is no last warp and no n or m; the factors a_t, b_t come with the tokens.
+struct ScanIn {
+    const float *q, *k, *v;    // the first token's; a head's q and k start (h / shared) * d behind
+    long long ld;              // between tokens
+    int shared;                // heads that share one q and k
+    const float* gates;        // NORM: [T, 2 H] log gates (i, then f); else [T, H, 2] (a, b)
+};
+
+template <int RW, bool NORM>
+__global__ void __launch_bounds__((RW + (NORM ? 1 : 0)) * 32)
+mlstm_scan_kernel(ScanIn in, float* __restrict__ num, float* __restrict__ den, int H, int d, int dv,
+                  float* __restrict__ state, long long state_stride, long long state_off,
                   const int* __restrict__ slots, const int* __restrict__ cu_seqlens) {
     pdl_wait();
     pdl_launch_next();
@@ -99,18 +110,21 @@ mlstm_scan_kernel(const float* __restrict__ qkv, const float* __restrict__ gates
     constexpr int DP = RW * ML_ROWS;                  // rows, padded
     constexpr int NR = RW >= 2 ? RW / 2 : 1;          // rows of n a lane of the last warp holds
     constexpr int CH = ML_CHUNK;
+    static_assert(2 * CH <= 32, "a warp copies the factors of a chunk");
     constexpr int CW = ML_COLS;
     constexpr int BUF = CH * (2 * DP + CW);
+    constexpr int NWARPS = RW + (NORM ? 1 : 0);
+    const float* __restrict__ gates = in.gates;
     float* coef = sm + 2 * BUF;                       // [2][CH][2]: a, b
     float* psum = coef + 4 * CH;                      // [2][CH][RW][CW]
     const int b = blockIdx.z, h = blockIdx.y;
     const int t0 = cu_seqlens[b], t1 = cu_seqlens[b + 1];
     const int slot = slots[b];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const bool is_nw = warp == RW;
+    const bool is_nw = NORM && warp == RW;
     const int col = blockIdx.x * CW + lane;
     const bool live = col < dv;
-    const int nq = H * d, C = 2 * nq + H * dv;
+    const int hg = h / in.shared;
     if (slot < 0) {
         // a padding entry: its rows are written, with zeros
         for (int t = t0; t < t1; ++t) {
@@ -122,7 +136,7 @@ mlstm_scan_kernel(const float* __restrict__ qkv, const float* __restrict__ gates
         }
         return;
     }
-    float* st = state + (size_t)slot * state_stride;
+    float* st = state + (size_t)slot * state_stride + state_off;
     float* S_g = st + (size_t)h * d * dv;
     float* n_g = st + (size_t)H * d * dv + (size_t)h * d;
     float* m_g = st + (size_t)H * d * dv + (size_t)H * d + (size_t)h * mlstm_m_copies(dv) +
@@ -144,7 +158,7 @@ mlstm_scan_kernel(const float* __restrict__ qkv, const float* __restrict__ gates
     // the padding rows of both buffers stay zero
     for (int i = threadIdx.x; i < 2 * BUF; i += blockDim.x) sm[i] = 0.f;
     __syncthreads();
-    float m_in = *m_g;                                // (the last warp's)
+    float m_in = NORM ? *m_g : 0.f;                   // (the last warp's)
     const int n_chunks = (t1 - t0 + CH - 1) / CH;
     auto issue = [&](int c) {
         float* qs = sm + (c & 1) * BUF;
@@ -152,16 +166,18 @@ mlstm_scan_kernel(const float* __restrict__ qkv, const float* __restrict__ gates
         float* vs = ks + CH * DP;
         const int c0 = t0 + c * CH, nt = min(CH, t1 - c0);
         // a warp a token, lanes along the row: no division in the walk
-        for (int tt = warp; tt < nt; tt += RW + 1) {
-            const float* row = qkv + (size_t)(c0 + tt) * C + (size_t)h * d;
+        for (int tt = warp; tt < nt; tt += NWARPS) {
+            const size_t at = (size_t)(c0 + tt) * in.ld;
+            const float *qr = in.q + at + (size_t)hg * d, *kr = in.k + at + (size_t)hg * d;
             for (int r = lane; r < d; r += 32) {
-                cp_async4(qs + tt * DP + r, row + r);
-                cp_async4(ks + tt * DP + r, row + nq + r);
+                cp_async4(qs + tt * DP + r, qr + r);
+                cp_async4(ks + tt * DP + r, kr + r);
             }
-            if (live)
-                cp_async4(vs + tt * CW + lane,
-                          qkv + (size_t)(c0 + tt) * C + 2 * nq + (size_t)h * dv + col);
+            if (live) cp_async4(vs + tt * CW + lane, in.v + at + (size_t)h * dv + col);
         }
+        if (!NORM && warp == 0 && lane < 2 * nt)
+            cp_async4(coef + (c & 1) * CH * 2 + lane,
+                      gates + ((size_t)(c0 + lane / 2) * H + h) * 2 + (lane & 1));
         cp_async_commit();
     };
     // the last warp's lanes hold the gate logarithms of the chunk they turn into factors next
@@ -346,6 +362,39 @@ int row_in(RowIn<float>& in, const float* row, long long ld, const float* part, 
     return 0;
 }
 
+template <bool NORM>
+int launch_scan(const ScanIn& in, float* num, float* den, int B, int H, int d, int dv, float* state,
+                long long state_stride, long long state_off, const int* slots,
+                const int* cu_seqlens, cudaStream_t stream) {
+    int RW = 1;
+    while (RW * ML_ROWS < d) RW *= 2;
+    const dim3 grid((unsigned)((dv + ML_COLS - 1) / ML_COLS), (unsigned)H, (unsigned)B);
+    const size_t smem = ((size_t)2 * ML_CHUNK * (2 * RW * ML_ROWS + ML_COLS) + 4 * ML_CHUNK +
+                         (size_t)2 * ML_CHUNK * RW * ML_COLS) * sizeof(float);
+#define AGV_SCAN(RR)                                                                          \
+    do {                                                                                      \
+        auto kern = mlstm_scan_kernel<RR, NORM>;                                              \
+        static bool configured = false;          /* (the size follows from RR alone) */       \
+        if (smem > 48 * 1024 && !configured) {                                                \
+            AGV_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, \
+                                             (int)smem));                                     \
+            configured = true;                                                                \
+        }                                                                                     \
+        agv_launch_after(kern, grid, (RR + (NORM ? 1 : 0)) * 32, smem, stream, in, num, den, H, \
+                         d, dv, state, state_stride, state_off, slots, cu_seqlens);           \
+    } while (0)
+    switch (RW) {
+        case 1: AGV_SCAN(1); break;
+        case 2: AGV_SCAN(2); break;
+        case 4: AGV_SCAN(4); break;
+        case 8: AGV_SCAN(8); break;
+        default: AGV_SCAN(16); break;
+    }
+#undef AGV_SCAN
+    AGV_LAUNCH_OK("mlstm_scan_kernel");
+    return 0;
+}
+
 }  // namespace
 
 AGV_API int agv_mlstm_prepare(const float* row, long long ld, const float* part, int n_splits,
@@ -377,33 +426,28 @@ AGV_API int agv_mlstm_scan(const float* qkv, const float* gates, float* num, flo
     AGV_REQUIRE(state_stride >= agv_mlstm_state_numel(H, d, dv), "mlstm_scan: state too small");
     AGV_REQUIRE(agv_aligned(den, 8), "mlstm_scan: den must be 8-byte aligned");
     if (T == 0) return 0;
-    int RW = 1;
-    while (RW * ML_ROWS < d) RW *= 2;
-    const dim3 grid((unsigned)((dv + ML_COLS - 1) / ML_COLS), (unsigned)H, (unsigned)B);
-    const size_t smem = ((size_t)2 * ML_CHUNK * (2 * RW * ML_ROWS + ML_COLS) + 4 * ML_CHUNK +
-                         (size_t)2 * ML_CHUNK * RW * ML_COLS) * sizeof(float);
-#define AGV_SCAN(RR)                                                                          \
-    do {                                                                                      \
-        auto kern = mlstm_scan_kernel<RR>;                                                    \
-        static bool configured = false;          /* (the size follows from RR alone) */       \
-        if (smem > 48 * 1024 && !configured) {                                                \
-            AGV_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, \
-                                             (int)smem));                                     \
-            configured = true;                                                                \
-        }                                                                                     \
-        agv_launch_after(kern, grid, (RR + 1) * 32, smem, stream, qkv, gates, num, den, H, d, \
-                         dv, state, state_stride, slots, cu_seqlens);                         \
-    } while (0)
-    switch (RW) {
-        case 1: AGV_SCAN(1); break;
-        case 2: AGV_SCAN(2); break;
-        case 4: AGV_SCAN(4); break;
-        case 8: AGV_SCAN(8); break;
-        default: AGV_SCAN(16); break;
-    }
-#undef AGV_SCAN
-    AGV_LAUNCH_OK("mlstm_scan_kernel");
-    return 0;
+    const ScanIn in{qkv, qkv + (size_t)H * d, qkv + (size_t)2 * H * d, 2LL * H * d + (long long)H * dv,
+                    1, gates};
+    return launch_scan<true>(in, num, den, B, H, d, dv, state, state_stride, 0, slots, cu_seqlens,
+                             stream);
+}
+
+// The scan without normaliser.  q, k: [T, groups * d] and v: [T, H * dv], 32-bit, with row stride
+// ld (parts of one row each); head h reads the q and k of group h / (H / groups); coef [T, H, 2]:
+// a_t, b_t; out [T, H * dv] receives S_t^T q_t; state: S [H, d, dv] per slot from state_off on.
+AGV_API int agv_head_scan(const float* q, const float* k, const float* v, long long ld,
+                          const float* coef, float* out, int T, int B, int H, int groups, int d,
+                          int dv, float* state, long long state_stride, long long state_off,
+                          const int* slots, const int* cu_seqlens, cudaStream_t stream) {
+    AGV_REQUIRE(T >= 0 && B > 0 && H > 0 && groups > 0 && H % groups == 0 && d > 0 && dv > 0,
+                "head_scan: bad sizes");
+    AGV_REQUIRE(d <= 256, "head_scan: state size %d exceeds 256", d);
+    AGV_REQUIRE(state && state_stride >= state_off + (long long)H * d * dv, "head_scan: state too small");
+    AGV_REQUIRE(B <= 65535 && H <= 65535, "head_scan: batch or head count exceeds the grid limit");
+    if (T == 0) return 0;
+    const ScanIn in{q, k, v, ld, H / groups, coef};
+    return launch_scan<false>(in, out, nullptr, B, H, d, dv, state, state_stride, state_off, slots,
+                              cu_seqlens, stream);
 }
 
 AGV_API int agv_mlstm_out(const float* num, const float* den, float den_eps, const float* row,

@@ -14,7 +14,9 @@
 // then q | k | v = nh * hd + nkv * hd + nkv * hdv wide), no kv heads at all (a layer that
 // attends to another layer's keys and values brings only queries), and a query
 // temperature: every q head is multiplied by 1 + coef * ln(floor((p + 1) / every) + 1) at
-// position p, in 32-bit, before it is rounded.
+// position p, in 32-bit, before it is rounded; biases of the projection, added first; pairs
+// (2i, 2i + 1) rotated instead of split halves; and every value head divided by its root mean
+// square before it is stored.
 #include "common.cuh"
 #include "cache_write.cuh"
 #include <type_traits>
@@ -26,6 +28,13 @@ struct QueryTemp {
 __device__ __forceinline__ float query_temp(const QueryTemp& qt, int p) {
     return 1.0f + qt.coef * logf((float)((p + 1) / qt.every + 1));
 }
+
+// What the general kernel does besides.
+struct QkExtras {
+    const float* bias;         // [row width] added to the projection, or null
+    int interleaved;           // pairs (2i, 2i + 1) of the rotated dimensions
+    float v_eps;               // >= 0: value heads over their root mean square (this eps)
+};
 
 constexpr int QK_WARPS = 4;
 constexpr int QK_MAX_HD = 1024;
@@ -43,7 +52,7 @@ qk_norm_rope_store_kernel(T* __restrict__ qkv, long long row_stride,
                           float eps, const float* __restrict__ cosv,
                           const float* __restrict__ sinv, int rotary_half,
                           const int* __restrict__ positions, CacheWrite cw, int hdv_,
-                          QueryTemp qt) {
+                          QueryTemp qt, QkExtras ex) {
     pdl_wait();
     pdl_launch_next();
     extern __shared__ float smem[];
@@ -74,6 +83,7 @@ qk_norm_rope_store_kernel(T* __restrict__ qkv, long long row_stride,
             c_page = cw.page_table[(size_t)c_slot * cw.max_pages + (c_pos % cw.cap) / cw.page];
     }
 
+    const float* bias = ex.bias ? ex.bias + head_at : nullptr;
     float ss = 0.f;
     if (part) {
         // the projection arrives as 32-bit partial sums over ranges of K
@@ -82,6 +92,13 @@ qk_norm_rope_store_kernel(T* __restrict__ qkv, long long row_stride,
         // ranges of K are added in order
         for (int e0 = 0; e0 < hd; e0 += 256) {
             float v[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+            if (bias) {
+#pragma unroll
+                for (int i = 0; i < 8; ++i) {
+                    const int e = e0 + lane + 32 * i;
+                    if (e < hd) v[i] = bias[e];
+                }
+            }
 #pragma unroll 2
             for (int sp = 0; sp < n_splits; ++sp) {
                 const float* row = ps + (size_t)sp * split_stride;
@@ -102,14 +119,18 @@ qk_norm_rope_store_kernel(T* __restrict__ qkv, long long row_stride,
         }
     } else {
         for (int e = lane; e < hd; e += 32) {
-            const float v = to_f32(src[e]);
+            const float v = to_f32(src[e]) + (bias ? bias[e] : 0.f);
             buf[e] = v;
             ss += v * v;
         }
     }
     if (!is_q && !is_k) {
-        // v head: stored as projected
-        if (part) {
+        // v head: stored as projected, or over its root mean square
+        if (ex.v_eps >= 0.f) {
+            const float r = 1.0f / sqrtf(warp_sum(ss) / (float)hd + ex.v_eps);
+            for (int e = lane; e < hd; e += 32) buf[e] *= r;
+        }
+        if (part || bias || ex.v_eps >= 0.f) {
             __syncwarp();
             for (int e = lane; e < hd; e += 32) src[e] = from_f32<T>(buf[e]);
         }
@@ -127,10 +148,12 @@ qk_norm_rope_store_kernel(T* __restrict__ qkv, long long row_stride,
         if (cosv) {
             const float* c = cosv + (size_t)t * rotary_half;
             const float* s = sinv + (size_t)t * rotary_half;
+            // the pair of angle e: (e, e + half), or neighbours
+            const int mul = ex.interleaved ? 2 : 1, mate = ex.interleaved ? 1 : rotary_half;
             for (int e = lane; e < rotary_half; e += 32) {
-                const float re = buf[e], im = buf[e + rotary_half];
-                buf[e] = re * c[e] - im * s[e];
-                buf[e + rotary_half] = re * s[e] + im * c[e];
+                const float re = buf[e * mul], im = buf[e * mul + mate];
+                buf[e * mul] = re * c[e] - im * s[e];
+                buf[e * mul + mate] = re * s[e] + im * c[e];
             }
         }
         __syncwarp();
@@ -461,6 +484,9 @@ static bool launch_qk_reg(T* qkv, long long row_stride, const float* part, int n
 // hdv: the value head size (the row is q | k | v with v heads of hdv; the value pool's rows
 // are nkv * hdv); nkv may be 0 (queries only).  qt_coef != 0: the query temperature
 // 1 + qt_coef * ln(floor((p + 1) / qt_every) + 1) multiplies every q head (needs positions).
+// bias: [row width] 32-bit, added to the projection first, or null; interleaved != 0: the pairs
+// (2i, 2i + 1) of the first rotary_dim dimensions turn; v_eps >= 0: value heads are divided by
+// sqrt(mean v^2 + v_eps).
 AGV_API int agv_qk_norm_rope_store_ex(void* qkv, int dtype, long long row_stride, const float* part,
                                       int n_splits, int n_tokens, int nh,
                                       int nkv, int hd, const float* wq, const float* wk, float eps,
@@ -470,13 +496,13 @@ AGV_API int agv_qk_norm_rope_store_ex(void* qkv, int dtype, long long row_stride
                                       const int* seq_index, int max_pages, int page, int cap,
                                       void* vt, long long vt_ld, const int* cu_seqlens, int n_seq,
                                       int max_len, int hdv, float qt_coef, int qt_every,
+                                      const float* bias, int interleaved, float v_eps,
                                       cudaStream_t stream) {
     AGV_REQUIRE(n_tokens >= 0 && nh > 0 && nkv >= 0 && hd > 0 && hdv > 0, "qk_norm_rope: bad sizes");
     AGV_REQUIRE(hd <= QK_MAX_HD && hdv <= QK_MAX_HD, "qk_norm_rope: head sizes %d, %d exceed %d",
                 hd, hdv, QK_MAX_HD);
     AGV_REQUIRE(qt_coef == 0.f || (qt_every > 0 && positions),
                 "qk_norm_rope: the query temperature needs positions and a period >= 1");
-    AGV_REQUIRE(!vt || hdv == hd, "qk_norm_rope: the transposed values need equal head sizes");
     AGV_REQUIRE(nkv > 0 || !k_pool, "qk_norm_rope: nothing to store without kv heads");
     AGV_REQUIRE(rotary_dim % 2 == 0 && rotary_dim <= hd, "qk_norm_rope: rotary_dim %d must be even "
                 "and at most head_dim %d", rotary_dim, hd);
@@ -500,14 +526,16 @@ AGV_API int agv_qk_norm_rope_store_ex(void* qkv, int dtype, long long row_stride
     const unsigned grid = (unsigned)((items + QK_WARPS - 1) / QK_WARPS);
     const size_t smem = (size_t)QK_WARPS * (hd > hdv ? hd : hdv) * sizeof(float);
     const int half = cosv ? rotary_dim / 2 : 0;
-    if (dtype == AGV_F32 &&
+    const QkExtras ex{bias, interleaved, v_eps};
+    const bool simple = !bias && !(interleaved && cosv) && v_eps < 0.f;
+    if (simple && dtype == AGV_F32 &&
         launch_qk_reg<float>((float*)qkv, row_stride, part, n_splits, split_stride, n_tokens, nh,
                              nkv, hd, wq, wk, eps, cosv, sinv, rotary_dim, positions, cw, vw, grid,
                              stream, hdv, qt)) {
         AGV_LAUNCH_OK("qk_norm_rope_store_reg_kernel");
         return 0;
     }
-    if (dtype == AGV_BF16 &&
+    if (simple && dtype == AGV_BF16 &&
         launch_qk_reg<__nv_bfloat16>((__nv_bfloat16*)qkv, row_stride, part, n_splits, split_stride,
                                      n_tokens, nh, nkv, hd, wq, wk, eps, cosv, sinv, rotary_dim,
                                      positions, cw, vw, grid, stream, hdv, qt)) {
@@ -516,10 +544,10 @@ AGV_API int agv_qk_norm_rope_store_ex(void* qkv, int dtype, long long row_stride
     }
     if (dtype == AGV_F32)
         agv_launch(qk_norm_rope_store_kernel<float>, grid, QK_WARPS * 32, smem, stream, (float*)qkv, row_stride, part, n_splits, split_stride, n_tokens, nh, nkv, hd, wq, wk,
-            eps, cosv, sinv, half, positions, cw, hdv, qt);
+            eps, cosv, sinv, half, positions, cw, hdv, qt, ex);
     else if (dtype == AGV_BF16)
         agv_launch(qk_norm_rope_store_kernel<__nv_bfloat16>, grid, QK_WARPS * 32, smem, stream, (__nv_bfloat16*)qkv, row_stride, part, n_splits, split_stride, n_tokens, nh, nkv, hd,
-            wq, wk, eps, cosv, sinv, half, positions, cw, hdv, qt);
+            wq, wk, eps, cosv, sinv, half, positions, cw, hdv, qt, ex);
     else
         return agv_fail(-1, "qk_norm_rope: unknown dtype %d", dtype);
     AGV_LAUNCH_OK("qk_norm_rope_store_kernel");
@@ -527,7 +555,7 @@ AGV_API int agv_qk_norm_rope_store_ex(void* qkv, int dtype, long long row_stride
         // the general kernel does not transpose: a kernel of its own reads the values
         // that the launch above wrote
         const __nv_bfloat16* v = (const __nv_bfloat16*)qkv + (size_t)(nh + nkv) * hd;
-        return agv_transpose_values(v, row_stride, vt, vt_ld, cu_seqlens, n_seq, max_len, nkv, hd,
+        return agv_transpose_values(v, row_stride, vt, vt_ld, cu_seqlens, n_seq, max_len, nkv, hdv,
                                     stream);
     }
     return 0;
@@ -546,5 +574,6 @@ AGV_API int agv_qk_norm_rope_store(void* qkv, int dtype, long long row_stride, c
     return agv_qk_norm_rope_store_ex(qkv, dtype, row_stride, part, n_splits, n_tokens, nh, nkv, hd,
                                      wq, wk, eps, cosv, sinv, rotary_dim, positions, k_pool, v_pool,
                                      page_table, slots, lens, seq_index, max_pages, page, cap, vt,
-                                     vt_ld, cu_seqlens, n_seq, max_len, hd, 0.f, 1, stream);
+                                     vt_ld, cu_seqlens, n_seq, max_len, hd, 0.f, 1, nullptr, 0, -1.f,
+                                     stream);
 }

@@ -490,7 +490,9 @@ def qk_norm_rope_store(qkv: torch.Tensor, n_heads: int, n_kv_heads: int, head_di
                        seq_index: Optional[torch.Tensor] = None, page: int = 0,
                        cap: int = 0, partial: Optional[torch.Tensor] = None,
                        vt: Optional[torch.Tensor] = None, cu_seqlens: Optional[torch.Tensor] = None,
-                       max_len: int = 0, value_dim: int = 0, q_temp=None) -> None:
+                       max_len: int = 0, value_dim: int = 0, q_temp=None,
+                       bias: Optional[torch.Tensor] = None, interleaved: bool = False,
+                       value_eps: Optional[float] = None) -> None:
     """In place on qkv [T, (nh + 2 nkv) * hd]: per-head norm of q and k, rotation,
     and (if pools are given) the store of k and v rows into the paged cache.
     ``partial`` [S, T, (nh + 2 nkv) * hd] (32-bit partial sums of the projection)
@@ -500,7 +502,9 @@ def qk_norm_rope_store(qkv: torch.Tensor, n_heads: int, n_kv_heads: int, head_di
     ``value_dim``: the size of a v head where it differs from head_dim (the row is then
     nh * hd + nkv * hd + nkv * value_dim wide); n_kv_heads may be 0 (queries alone).
     ``q_temp`` = (coef, every): every q head is multiplied by
-    1 + coef * ln(floor((p + 1) / every) + 1) at position p."""
+    1 + coef * ln(floor((p + 1) / every) + 1) at position p.  ``bias`` [W] (32-bit) is added to
+    the projection first; ``interleaved``: neighbouring dimensions turn as pairs, not split
+    halves; ``value_eps``: every value head is divided by sqrt(mean v^2 + value_eps)."""
     T = qkv.shape[0]
     n_splits = 0
     hdv = value_dim or head_dim
@@ -511,6 +515,9 @@ def qk_norm_rope_store(qkv: torch.Tensor, n_heads: int, n_kv_heads: int, head_di
         n_splits = partial.shape[0]
     assert qkv.stride(1) == 1
     _f32(wq, "wq"); _f32(wk, "wk"); _f32(cos, "cos"); _f32(sin, "sin")
+    if bias is not None:
+        _f32(bias, "bias"); _dense(bias, "bias")
+        assert bias.numel() == (n_heads + n_kv_heads) * head_dim + n_kv_heads * hdv
     for t, n in ((positions, "positions"), (page_table, "page_table"), (slots, "slots"),
                  (lens, "lens"), (seq_index, "seq_index")):
         _i32(t, n)
@@ -521,7 +528,7 @@ def qk_norm_rope_store(qkv: torch.Tensor, n_heads: int, n_kv_heads: int, head_di
     n_seq = 0
     if vt is not None:
         _dense(vt, "vt"); _i32(cu_seqlens, "cu_seqlens")
-        assert vt.dtype == torch.bfloat16 and vt.shape[0] == n_kv_heads * head_dim
+        assert vt.dtype == torch.bfloat16 and vt.shape[0] == n_kv_heads * hdv
         n_seq = cu_seqlens.numel() - 1
     with _span("qk_norm_rope", 2 * _nbytes(qkv) + _nbytes(partial, vt)):
         coef, every = q_temp if q_temp is not None else (0.0, 1)
@@ -531,7 +538,9 @@ def qk_norm_rope_store(qkv: torch.Tensor, n_heads: int, n_kv_heads: int, head_di
             _ptr(cos), _ptr(sin), rotary_dim, _ptr(positions), _ptr(k_pool), _ptr(v_pool),
             _ptr(page_table), _ptr(slots), _ptr(lens), _ptr(seq_index), max_pages, page, cap,
             _ptr(vt), ctypes.c_longlong(vt.shape[1] if vt is not None else 0), _ptr(cu_seqlens),
-            n_seq, max_len, hdv, ctypes.c_float(coef), int(every), _stream()))
+            n_seq, max_len, hdv, ctypes.c_float(coef), int(every), _ptr(bias),
+            1 if interleaved else 0, ctypes.c_float(-1.0 if value_eps is None else value_eps),
+            _stream()))
 
 
 _FUSED_QKV = os.environ.get("AGAVE_B200_FUSED_QKV_PREFILL", "1") != "0"
@@ -603,11 +612,12 @@ def attention_prefill_simt(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, ou
                            scale: float, window: int, value_dim: int = 0,
                            sinks: Optional[torch.Tensor] = None,
                            dist_bias: Optional[torch.Tensor] = None,
-                           keep_first: int = 0) -> None:
+                           keep_first: int = 0, softcap: float = 0.0) -> None:
     """Prompts that start at 0; q [T, nh*hd], k [T, nkv*hd], v [T, nkv*hdv] row-strided
     views (hdv = value_dim or head_dim), out [T, nh*hdv]; ``sinks`` [nh]: a logit per query
     head that joins its softmax denominator once; ``dist_bias`` [nh, n]: added to the scaled
-    score of a key at distance min(t - j, n - 1)."""
+    score of a key at distance min(t - j, n - 1); ``softcap`` > 0: the scaled score s becomes
+    softcap * tanh(s / softcap) (before the bias)."""
     T = q.shape[0]
     assert q.stride(1) == 1 and k.stride(1) == 1 and v.stride(1) == 1
     _dense(out, "out"); _f32(sinks, "sinks"); _f32(dist_bias, "dist_bias")
@@ -621,7 +631,7 @@ def attention_prefill_simt(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, ou
         _ptr(seq_index), _ptr(cu_seqlens), T, n_heads, n_kv_heads, head_dim,
         ctypes.c_float(scale), window, value_dim or head_dim, ctypes.c_longlong(v.stride(0)),
         _ptr(sinks), _ptr(dist_bias), dist_bias.shape[1] if dist_bias is not None else 0,
-        int(keep_first), _stream()))
+        int(keep_first), ctypes.c_float(softcap), _stream()))
 
 
 def attention_paged_simt(q: torch.Tensor, out: torch.Tensor, k_pool: torch.Tensor,
@@ -631,7 +641,7 @@ def attention_paged_simt(q: torch.Tensor, out: torch.Tensor, k_pool: torch.Tenso
                          window: int, value_dim: int = 0,
                          sinks: Optional[torch.Tensor] = None,
                          dist_bias: Optional[torch.Tensor] = None, v_row: int = 0,
-                         keep_first: int = 0) -> None:
+                         keep_first: int = 0, softcap: float = 0.0) -> None:
     """Queries against the paged cache; their own keys are already stored.  ``v_row``: the
     elements between two positions' value rows where that is not nkv * hdv (values that are
     the leading part of the key rows: v_pool is then k_pool)."""
@@ -652,7 +662,7 @@ def attention_paged_simt(q: torch.Tensor, out: torch.Tensor, k_pool: torch.Tenso
         page_table.shape[1], page, cap, T, n_heads, n_kv_heads, head_dim,
         ctypes.c_float(scale), window, value_dim or head_dim, _ptr(sinks), _ptr(dist_bias),
         dist_bias.shape[1] if dist_bias is not None else 0, int(v_row), int(keep_first),
-        _stream()))
+        ctypes.c_float(softcap), _stream()))
 
 
 # ------------------------------------------- rows of stacked projections, latent attention
@@ -978,6 +988,188 @@ def mlstm_out(num: torch.Tensor, den: torch.Tensor, den_eps: float, row: Optiona
         _check(library().agv_mlstm_out(_ptr(num), _ptr(den), ctypes.c_float(den_eps), rp, ld, pp,
                                        ns, _ptr(weight), ctypes.c_float(eps), T, H, d, dv,
                                        _ptr(y), dtype_code(y.dtype), _stream()))
+
+
+# ------------------------------------------------------- state-space mixers
+def ssm_conv(row: Optional[torch.Tensor], partial: Optional[torch.Tensor], T: int, W: int,
+             offset: int, taps: int, conv_w: torch.Tensor, conv_b: torch.Tensor,
+             out: torch.Tensor, rounded: Optional[torch.Tensor], state: torch.Tensor,
+             state_off: int, ctx, dt_offset: int = 0, dt_bias: Optional[torch.Tensor] = None,
+             neg_a: Optional[torch.Tensor] = None, coef: Optional[torch.Tensor] = None) -> None:
+    """From channels ``offset`` .. of a token's row of the stacked projection (32-bit rows [T, W]
+    or ``partial`` [S, T, W]): a causal convolution over ``taps`` tokens per channel with a bias,
+    then silu, into out [T, C] (32-bit) and, if given, ``rounded`` [T, C] (another dtype).
+    Earlier inputs come from the step's rows or from the ring in ``state`` at ``state_off``,
+    which is brought up to date.  With ``coef`` [T, H, 2]: the columns ``dt_offset`` .. + H are
+    step sizes, dt = softplus(x + dt_bias), and coef receives (exp(neg_a * dt), dt)."""
+    rp, ld, pp, ns = _f32_row_input(row, partial, T, W)
+    C = conv_w.shape[0]
+    for t, n in ((conv_w, "conv_w"), (conv_b, "conv_b"), (out, "out"), (dt_bias, "dt_bias"),
+                 (neg_a, "neg_a"), (coef, "coef")):
+        _f32(t, n)
+        if t is not None:
+            _dense(t, n)
+    assert conv_w.shape == (C, taps) and conv_b.numel() == C and out.shape == (T, C)
+    n_dt = 0
+    if coef is not None:
+        n_dt = dt_bias.numel()
+        assert neg_a.numel() == n_dt and coef.shape == (T, n_dt, 2)
+    if rounded is not None:
+        _dense(rounded, "rounded")
+        assert rounded.shape == (T, C)
+    if state is not None:
+        sp, ss = _state_args(state)
+    else:
+        sp, ss = ctypes.c_void_p(0), ctypes.c_longlong(0)
+    with _span("ssm_conv", _nbytes(out, rounded, coef) + T * (C + n_dt) * 4 * max(ns, 1)):
+        _check(library().agv_ssm_conv(
+            rp, ld, pp, ns, T, W, offset, C, taps, _ptr(conv_w), _ptr(conv_b), _ptr(out),
+            _ptr(rounded), dtype_code(rounded.dtype) if rounded is not None else F32, dt_offset,
+            n_dt, _ptr(dt_bias), _ptr(neg_a), _ptr(coef), sp, ss, ctypes.c_longlong(state_off),
+            _ptr(ctx.slots), _ptr(ctx.cu_seqlens), _ptr(ctx.seq_index), _ptr(ctx.positions),
+            _ptr(ctx.lens), _stream()))
+
+
+SELECTIVE_MAX_STATE = 256
+
+
+def selective_pad(n_state: int) -> int:
+    """The states of a channel as the selective scan pads them: 4, 8, 16 .. 256."""
+    n = 4
+    while n < n_state:
+        n *= 2
+    return n
+
+
+def selective_low(row: Optional[torch.Tensor], partial: Optional[torch.Tensor], dt_rank: int,
+                  n_state: int, low: torch.Tensor, bc: torch.Tensor) -> None:
+    """From a row  r | B | C  of the second projection (compute dtype, or 32-bit partial sums):
+    low [T, dt_rank] = r in the compute dtype, bc [T, 2 * pad] = B and C, 32-bit, each padded
+    with zeros to ``selective_pad(n_state)``."""
+    T = low.shape[0]
+    rp, ld, pp, ns = _row_input(row, partial, T, dt_rank + 2 * n_state)
+    _dense(low, "low"); _dense(bc, "bc"); _f32(bc, "bc")
+    assert low.shape == (T, dt_rank) and bc.shape == (T, 2 * selective_pad(n_state))
+    assert row is None or row.dtype == low.dtype
+    with _span("selective_low", _nbytes(row, partial, low, bc)):
+        _check(library().agv_selective_low(rp, ctypes.c_longlong(ld), pp, ns, dtype_code(low.dtype),
+                                           T, dt_rank, n_state, _ptr(low), _ptr(bc), _stream()))
+
+
+def selective_scan(u: torch.Tensor, dt: torch.Tensor, dt_bias: torch.Tensor, bc: torch.Tensor,
+                   a2: torch.Tensor, d: torch.Tensor, row: Optional[torch.Tensor],
+                   partial: Optional[torch.Tensor], W: int, z_offset: int, out: torch.Tensor, ctx,
+                   state: torch.Tensor, state_off: int) -> None:
+    """S[c, n] <- exp(dt_c A[c, n]) S[c, n] + dt_c u_c B_n;  y_c = sum_n S[c, n] C_n + D_c u_c  over
+    the step's tokens, sequence by sequence, with dt_c = softplus(dt_c + dt_bias_c) and ``a2`` =
+    A * log2(e); out = y * silu(z), z the columns ``z_offset`` .. of the stacked projection.  S
+    [inner, N] of each sequence is read from and written to ``state`` at ``state_off``."""
+    T, inner = u.shape
+    N = a2.shape[1]
+    rp, ld, pp, ns = _f32_row_input(row, partial, T, W)
+    for t, n in ((u, "u"), (dt, "dt"), (dt_bias, "dt_bias"), (bc, "bc"), (a2, "a2"), (d, "d")):
+        _f32(t, n); _dense(t, n)
+    _dense(out, "out")
+    assert dt.shape == (T, inner) and out.shape == (T, inner) and a2.shape[0] == inner
+    assert bc.shape == (T, 2 * selective_pad(N)) and dt_bias.numel() == inner and d.numel() == inner
+    lib = library()
+    assert lib.agv_selective_pad(N) == selective_pad(N)
+    sp, ss = _state_args(state)
+    with _span("selective_scan", _nbytes(u, dt, bc, out) + T * inner * 4 * max(ns, 1) +
+               8 * ctx.batch * inner * N, 7 * T * inner * N):
+        _check(lib.agv_selective_scan(
+            _ptr(u), _ptr(dt), _ptr(dt_bias), _ptr(bc), _ptr(a2), _ptr(d), rp, ld, pp, ns, T, W,
+            z_offset, ctx.batch, inner, N, _ptr(out), dtype_code(out.dtype), sp, ss,
+            ctypes.c_longlong(state_off), _ptr(ctx.slots), _ptr(ctx.cu_seqlens), _stream()))
+
+
+def head_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, coef: torch.Tensor,
+              out: torch.Tensor, ctx, state: torch.Tensor, state_off: int, n_heads: int,
+              n_groups: int, state_dim: int, value_dim: int) -> None:
+    """S <- a S + b k v^T;  o = S^T q  per head over the step's tokens, sequence by sequence, with
+    (a, b) = coef[t, h]; q, k [T, n_groups * state_dim] and v [T, n_heads * value_dim] are column
+    ranges of one 32-bit tensor, head h reads the q and k of group h // (n_heads / n_groups).  S
+    [H, state_dim, value_dim] of each sequence is in ``state`` at ``state_off``."""
+    T = v.shape[0]
+    H, N, dv = n_heads, state_dim, value_dim
+    for t, n in ((q, "q"), (k, "k"), (v, "v"), (coef, "coef"), (out, "out")):
+        _f32(t, n)
+    assert q.shape == k.shape == (T, n_groups * N) and v.shape == (T, H * dv)
+    assert q.stride(0) == k.stride(0) == v.stride(0) and q.stride(1) == v.stride(1) == 1
+    _dense(coef, "coef"); _dense(out, "out")
+    assert coef.shape == (T, H, 2) and out.shape == (T, H * dv)
+    sp, ss = _state_args(state)
+    with _span("head_scan", _nbytes(q, k, v, coef, out) + 8 * ctx.batch * H * N * dv,
+               5 * T * H * N * dv):
+        _check(library().agv_head_scan(
+            _ptr(q), _ptr(k), _ptr(v), ctypes.c_longlong(v.stride(0)), _ptr(coef), _ptr(out), T,
+            ctx.batch, H, n_groups, N, dv, sp, ss, ctypes.c_longlong(state_off), _ptr(ctx.slots),
+            _ptr(ctx.cu_seqlens), _stream()))
+
+
+def ssd_out(num: torch.Tensor, u: torch.Tensor, d: torch.Tensor, row: Optional[torch.Tensor],
+            partial: Optional[torch.Tensor], W: int, z_offset: int, weight: torch.Tensor,
+            eps: float, n_parts: int, value_dim: int, y: torch.Tensor) -> None:
+    """y = g / rms(g) * weight with g = (num + D_h u) * silu(z), the root mean square taken over
+    each of ``n_parts`` equal parts of the row; z: columns ``z_offset`` .. of the stacked
+    projection; ``u``: a column range of a 32-bit tensor."""
+    T, inner = num.shape
+    rp, ld, pp, ns = _f32_row_input(row, partial, T, W)
+    for t, n in ((num, "num"), (d, "d"), (weight, "weight")):
+        _f32(t, n); _dense(t, n)
+    _f32(u, "u"); _dense(y, "y")
+    assert u.shape == (T, inner) and u.stride(1) == 1 and y.shape == (T, inner)
+    assert weight.numel() == inner and d.numel() * value_dim == inner
+    with _span("ssd_out", _nbytes(num, u, y) + T * inner * 4 * max(ns, 1)):
+        _check(library().agv_ssd_out(
+            _ptr(num), _ptr(u), ctypes.c_longlong(u.stride(0)), _ptr(d), rp, ld, pp, ns, T, W,
+            z_offset, _ptr(weight), ctypes.c_float(eps), inner, value_dim, n_parts, _ptr(y),
+            dtype_code(y.dtype), _stream()))
+
+
+def gated_join(h: Optional[torch.Tensor], terms, gate_row: Optional[torch.Tensor],
+               gate_partial: Optional[torch.Tensor], gate_bias: Optional[torch.Tensor],
+               w_next: Optional[torch.Tensor], eps: float, x: Optional[torch.Tensor]) -> None:
+    """Several branches join the 32-bit stream h [R, H] in one launch:
+    h += sum_i mult_i * sigmoid(logits[gate_i] + bias[gate_i]) * y_i, then x = rmsnorm(h) * w_next
+    if there is one (x alone: the sum as it is; h None: the sum starts at zero).
+
+    ``terms``: (y, mult, gate) with y [R, H] or 32-bit partial sums [S, R, H] and gate the index
+    of its gate or -1; the gates' logits are stacked, 32-bit [R, G * H] or [S, R, G * H]."""
+    first = terms[0][0]
+    R, H = first.shape[-2:]
+    n = len(terms)
+    ys, dts, splits = (ctypes.c_void_p * n)(), (ctypes.c_int * n)(), (ctypes.c_int * n)()
+    mults, gates = (ctypes.c_float * n)(), (ctypes.c_int * n)()
+    for i, (y, mult, gate) in enumerate(terms):
+        _dense(y, "y")
+        assert y.shape[-2:] == (R, H)
+        if y.dim() == 3:
+            _f32(y, "y")
+        ys[i], dts[i] = _ptr(y), dtype_code(y.dtype)
+        splits[i] = y.shape[0] if y.dim() == 3 else 1
+        mults[i], gates[i] = float(mult), int(gate)
+    n_gates = 0
+    rp, ld = ctypes.c_void_p(0), ctypes.c_longlong(0)
+    pp, gs = ctypes.c_void_p(0), 0
+    if gate_bias is not None:
+        _f32(gate_bias, "gate_bias"); _dense(gate_bias, "gate_bias")
+        assert gate_bias.numel() % H == 0
+        n_gates = gate_bias.numel() // H
+        rp, ld, pp, gs = _f32_row_input(gate_row, gate_partial, R, n_gates * H)
+    if h is not None:
+        _f32(h, "h"); _dense(h, "h")
+        assert h.shape == (R, H)
+    _f32(w_next, "w_next")
+    if x is not None:
+        _dense(x, "x")
+        assert x.shape == (R, H)
+    with _span("norm", _nbytes(*[t[0] for t in terms], gate_row, gate_partial, x) +
+               (R * H * 8 if h is not None else 0)):
+        _check(library().agv_gated_join(
+            _ptr(h), R, H, n, ys, dts, splits, mults, gates, n_gates, rp, ld, pp, gs,
+            _ptr(gate_bias), _ptr(w_next), ctypes.c_float(eps), _ptr(x),
+            dtype_code(x.dtype) if x is not None else F32, _stream()))
 
 
 # ------------------------------------------- attention with a short convolution
@@ -1343,7 +1535,8 @@ def attention_prefill_mma(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, out
                           cu_seqlens: torch.Tensor, max_len: int, n_heads: int, n_kv_heads: int,
                           head_dim: int, scale: float, window: int,
                           sinks: Optional[torch.Tensor] = None, value_dim: int = 0,
-                          dist_bias: Optional[torch.Tensor] = None, keep_first: int = 0) -> None:
+                          dist_bias: Optional[torch.Tensor] = None, keep_first: int = 0,
+                          softcap: float = 0.0) -> None:
     """Prompts that start at 0 on the tensor cores (bfloat16, head sizes in steps
     of 8 up to 256); q, k, v are row-strided views, out is dense.  ``value_dim``: the value
     head size where it differs from the keys'; ``dist_bias`` [nh, n]: see
@@ -1360,7 +1553,8 @@ def attention_prefill_mma(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, out
         ctypes.c_longlong(k.stride(0)), _ptr(out), _ptr(cu_seqlens), cu_seqlens.numel() - 1,
         max_len, n_heads, n_kv_heads, head_dim, ctypes.c_float(scale), window, _ptr(sinks),
         value_dim or head_dim, ctypes.c_longlong(v.stride(0)), _ptr(dist_bias),
-        dist_bias.shape[1] if dist_bias is not None else 0, int(keep_first), _stream()))
+        dist_bias.shape[1] if dist_bias is not None else 0, int(keep_first),
+        ctypes.c_float(softcap), _stream()))
 
 
 def prefill_values_scratch(T: int, B: int, n_kv_heads: int, head_dim: int,
@@ -1387,20 +1581,22 @@ def attention_prefill_tc(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, out:
                          head_dim: int, scale: float, window: int,
                          vt: Optional[torch.Tensor] = None,
                          sinks: Optional[torch.Tensor] = None,
-                         dist_bias: Optional[torch.Tensor] = None, keep_first: int = 0) -> None:
-    """Prompts that start at 0 on the tcgen05 tensor cores (bfloat16, head sizes in
-    steps of 16 up to 256); q, k, v are row-strided views, out is dense.  ``vt``:
+                         dist_bias: Optional[torch.Tensor] = None, keep_first: int = 0,
+                         value_dim: int = 0, softcap: float = 0.0) -> None:
+    """Prompts that start at 0 on the tcgen05 tensor cores (bfloat16, key and value head
+    sizes in steps of 16 up to 256); q, k, v are row-strided views, out is dense.  ``vt``:
     the values already transposed (by ``qk_norm_rope_store``); else this call
     transposes them."""
     assert q.dtype == torch.bfloat16 and k.dtype == q.dtype and v.dtype == q.dtype
     assert q.stride(1) == 1 and k.stride(1) == 1 and v.stride(1) == 1
-    assert k.stride(0) == v.stride(0)
     _dense(out, "out"); _i32(cu_seqlens, "cu_seqlens")
     T, B = q.shape[0], cu_seqlens.numel() - 1
+    hdv = value_dim or head_dim
     ready = vt is not None
     if vt is None:
-        vt = prefill_values_scratch(T, B, n_kv_heads, head_dim, q.device)
+        vt = prefill_values_scratch(T, B, n_kv_heads, hdv, q.device)
     _dense(vt, "vt")
+    assert vt.shape[0] == n_kv_heads * hdv
     _f32(sinks, "sinks"); _f32(dist_bias, "dist_bias")
     if dist_bias is not None:
         _dense(dist_bias, "dist_bias")
@@ -1410,7 +1606,8 @@ def attention_prefill_tc(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, out:
         ctypes.c_longlong(k.stride(0)), _ptr(out), _ptr(vt), ctypes.c_longlong(vt.shape[1]),
         1 if ready else 0, _ptr(cu_seqlens), B, T, max_len, n_heads, n_kv_heads, head_dim,
         ctypes.c_float(scale), window, _ptr(sinks), _ptr(dist_bias),
-        dist_bias.shape[1] if dist_bias is not None else 0, int(keep_first), _stream()))
+        dist_bias.shape[1] if dist_bias is not None else 0, int(keep_first), hdv,
+        ctypes.c_longlong(v.stride(0)), ctypes.c_float(softcap), _stream()))
 
 
 def attention_tc_status() -> int:
@@ -1431,40 +1628,42 @@ def attention_prefill_wants_transposed_values(qkv: torch.Tensor, head_dim: int,
                                               value_dim: int = 0) -> bool:
     """Whether ``attention_prefill`` on views of this projection output will take the
     tcgen05 kernel, which reads the values transposed."""
-    return ((value_dim or head_dim) == head_dim and _PREFILL_TC and qkv.shape[0] > PREFILL_TC_MIN_TOKENS and qkv.dtype == torch.bfloat16 and
-            head_dim % 16 == 0 and head_dim <= 256 and qkv.stride(0) % 8 == 0 and
-            qkv.data_ptr() % 16 == 0)
+    hdv = value_dim or head_dim
+    return (_PREFILL_TC and qkv.shape[0] > PREFILL_TC_MIN_TOKENS and qkv.dtype == torch.bfloat16 and
+            head_dim % 16 == 0 and head_dim <= 256 and hdv % 16 == 0 and hdv <= 256 and
+            qkv.stride(0) % 8 == 0 and qkv.data_ptr() % 16 == 0)
 
 
 def attention_prefill(q, k, v, out, ctx, n_heads, n_kv_heads, head_dim, scale, window,
                       vt=None, value_dim: int = 0, sinks=None, dist_bias=None,
-                      op: str = "attention", keep_first: int = 0) -> None:
-    """Prompt attention of one layer in bfloat16: the tcgen05 kernel for head sizes
-    in steps of 16 up to 256, the mma.sync kernel for the other multiples of 8; else
-    (and for value heads of another size than the keys') the one-warp-per-(token, head)
-    kernel.  ``sinks`` [nh]: a logit per query head that joins its denominator once."""
+                      op: str = "attention", keep_first: int = 0, softcap: float = 0.0) -> None:
+    """Prompt attention of one layer in bfloat16: the tcgen05 kernel for key and value head
+    sizes in steps of 16 up to 256, the mma.sync kernel for the other multiples of 8; else
+    the one-warp-per-(token, head) kernel.  ``sinks`` [nh]: a logit per query head that joins its denominator once."""
     hdv = value_dim or head_dim
     aligned = (q.dtype == torch.bfloat16 and head_dim <= 256 and hdv <= 256 and
                q.stride(0) % 8 == 0 and k.stride(0) % 8 == 0 and v.stride(0) % 8 == 0 and
                q.data_ptr() % 16 == 0 and k.data_ptr() % 16 == 0 and v.data_ptr() % 16 == 0)
-    # the tcgen05 kernel does not know value heads of their own size
-    same = hdv == head_dim and k.stride(0) == v.stride(0)
+    # (the tcgen05 kernel has a form with a distance bias and one with a soft cap, none with both)
+    tc = head_dim % 16 == 0 and hdv % 16 == 0 and not (softcap and dist_bias is not None)
     if not window:
         keep_first = 0                    # (without a window every key is visible anyway)
     with _span(op, *_attention_cost(ctx, q, k, v, out, n_heads, head_dim, window)):
-        if (aligned and same and head_dim % 16 == 0 and _PREFILL_TC and scale > 0 and
+        if (aligned and tc and _PREFILL_TC and scale > 0 and
                 q.shape[0] > PREFILL_TC_MIN_TOKENS):
             attention_prefill_tc(q, k, v, out, ctx.cu_seqlens, ctx.max_new, n_heads, n_kv_heads,
                                  head_dim, scale, window, vt=vt, sinks=sinks, dist_bias=dist_bias,
-                                 keep_first=keep_first)
+                                 keep_first=keep_first, value_dim=hdv, softcap=softcap)
         elif aligned and head_dim % 8 == 0 and hdv % 8 == 0:
             attention_prefill_mma(q, k, v, out, ctx.cu_seqlens, ctx.max_new, n_heads,
                                   n_kv_heads, head_dim, scale, window, sinks=sinks,
-                                  value_dim=hdv, dist_bias=dist_bias, keep_first=keep_first)
+                                  value_dim=hdv, dist_bias=dist_bias, keep_first=keep_first,
+                                  softcap=softcap)
         else:
             attention_prefill_simt(q, k, v, out, ctx.positions, ctx.seq_index, ctx.cu_seqlens,
                                    n_heads, n_kv_heads, head_dim, scale, window, value_dim=hdv,
-                                   sinks=sinks, dist_bias=dist_bias, keep_first=keep_first)
+                                   sinks=sinks, dist_bias=dist_bias, keep_first=keep_first,
+                                   softcap=softcap)
 
 
 def _attention_cost(ctx, q, k, v, out, n_heads, head_dim, window, n_kv_heads=0):
@@ -1546,7 +1745,8 @@ def attention_decode_split(q: torch.Tensor, out: torch.Tensor, k_pool: torch.Ten
                            max_keys: int, part_acc: Optional[torch.Tensor] = None,
                            part_ml: Optional[torch.Tensor] = None,
                            sinks: Optional[torch.Tensor] = None,
-                           dist_bias: Optional[torch.Tensor] = None, keep_first: int = 0) -> None:
+                           dist_bias: Optional[torch.Tensor] = None, keep_first: int = 0,
+                           value_dim: int = 0, softcap: float = 0.0) -> None:
     """One query per batch entry against the paged cache, keys split into chunks
     whose partial results go through scratch memory (allocated here if not given)."""
     B = q.shape[0]
@@ -1555,12 +1755,14 @@ def attention_decode_split(q: torch.Tensor, out: torch.Tensor, k_pool: torch.Ten
     for t, n in ((positions, "positions"), (page_table, "page_table"), (slots, "slots")):
         _i32(t, n)
     assert k_pool.dtype == q.dtype and out.dtype == q.dtype
-    _, n_splits = attention_decode_plan(head_dim, q.dtype, max_keys)
+    hdv = value_dim or head_dim
+    _, n_splits = attention_decode_plan(max(head_dim, hdv), q.dtype, max_keys)
     if part_acc is None:
-        part_acc = torch.empty((B, n_heads, n_splits, head_dim), dtype=torch.float32,
+        part_acc = torch.empty((B, n_heads, n_splits, hdv), dtype=torch.float32,
                                device=q.device)
         part_ml = torch.empty((B, n_heads, n_splits, 2), dtype=torch.float32, device=q.device)
-    assert part_acc.numel() >= B * n_heads * n_splits * head_dim
+    assert part_acc.numel() >= B * n_heads * n_splits * hdv
+    assert out.numel() == B * n_heads * hdv
     assert part_ml.numel() >= B * n_heads * n_splits * 2
     _f32(part_acc, "part_acc"); _f32(part_ml, "part_ml")
     counters = _decode_counters(q.device, B * n_heads)
@@ -1573,7 +1775,8 @@ def attention_decode_split(q: torch.Tensor, out: torch.Tensor, k_pool: torch.Ten
         _ptr(v_pool), _ptr(page_table), _ptr(slots), _ptr(positions), page_table.shape[1], page,
         cap, B, n_heads, n_kv_heads, head_dim, ctypes.c_float(scale), window, max_keys,
         _ptr(part_acc), _ptr(part_ml), _ptr(counters), _ptr(sinks), _ptr(dist_bias),
-        dist_bias.shape[1] if dist_bias is not None else 0, int(keep_first), _stream()))
+        dist_bias.shape[1] if dist_bias is not None else 0, int(keep_first), hdv,
+        ctypes.c_float(softcap), _stream()))
 
 
 _FUSED_DECODE = os.environ.get("AGAVE_B200_FUSED_DECODE_ATTENTION", "1") != "0"
@@ -1631,27 +1834,28 @@ def attention_decode_fused(partial: torch.Tensor, wq: Optional[torch.Tensor],
 def attention_decode(q, out, view, ctx, n_heads, n_kv_heads, head_dim, scale, window,
                      value_dim: int = 0, sinks=None, dist_bias=None,
                      values_in_keys: bool = False, op: str = "attention",
-                     keep_first: int = 0) -> None:
-    """Decode attention of one layer: the split kernel for head sizes in steps of
-    16 up to 512, else (and for value heads of another size than the keys') the
-    one-warp-per-head kernel."""
+                     keep_first: int = 0, softcap: float = 0.0) -> None:
+    """Decode attention of one layer: the split kernel for key and value head sizes in steps
+    of 16 up to 512, else the one-warp-per-head kernel."""
     hdv = value_dim or head_dim
     if not window:
         keep_first = 0
     with _span(op, *_attention_cost(ctx, q, None, None, out, n_heads, head_dim, window,
                                     n_kv_heads)):
-        if (head_dim % 16 == 0 and head_dim <= 512 and hdv == head_dim and not values_in_keys
+        if (head_dim % 16 == 0 and head_dim <= 512 and hdv % 16 == 0 and hdv <= 512
+                and not values_in_keys
                 and not (keep_first and dist_bias is not None)):
             # (kept first keys are walked before the window's)
             max_keys = min(abs(window) + keep_first, ctx.max_len) if window else ctx.max_len
             attention_decode_split(q, out, view.k_pool, view.v_pool, view.page_table, ctx.slots,
                                    ctx.positions, view.page, view.cap, n_heads, n_kv_heads,
                                    head_dim, scale, window, max(1, max_keys), sinks=sinks,
-                                   dist_bias=dist_bias, keep_first=keep_first)
+                                   dist_bias=dist_bias, keep_first=keep_first, value_dim=hdv,
+                                   softcap=softcap)
         else:
             attention_paged_simt(q, out, view.k_pool, view.v_pool, view.page_table, ctx.slots,
                                  ctx.positions, ctx.seq_index, view.page, view.cap, n_heads,
                                  n_kv_heads, head_dim, scale, window, value_dim=hdv, sinks=sinks,
                                  dist_bias=dist_bias,
                                  v_row=n_kv_heads * head_dim if values_in_keys else 0,
-                                 keep_first=keep_first)
+                                 keep_first=keep_first, softcap=softcap)

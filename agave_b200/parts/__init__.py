@@ -11,6 +11,8 @@ from .position import LearnedPosition
 from .feedforward import DenseFeedForward, GatedFeedForward
 from .moe import RoutedFeedForward
 from .block import Block
+from .state_space import SelectiveScanMixer, StateSpaceMixer
+from .parallel import ParallelBlock, SideBySideMixer
 from .linear import GatedLinear, Linear
 
 __all__ = ["KVRequest", "ParamSpec", "StateRequest", "feed_forward_class", "mixer_class",
@@ -19,4 +21,5 @@ __all__ = ["KVRequest", "ParamSpec", "StateRequest", "feed_forward_class", "mixe
            "register_position", "register_stream_position", "RMSNorm", "LayerNorm",
            "RoutedFeedForward", "RotaryEmbedding", "Identity", "LatentAttentionMixer",
            "DenseFeedForward", "ChannelDeltaMixer", "LearnedPosition",
+           "SelectiveScanMixer", "StateSpaceMixer", "ParallelBlock", "SideBySideMixer",
            "AttentionMixer", "GatedFeedForward", "Block", "GatedLinear", "Linear"]

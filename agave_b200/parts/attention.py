@@ -39,7 +39,11 @@ key); a short causal convolution over time on every channel of q, k and v, betwe
 projection and the rotation (``conv_taps``; tensors ``q_conv.weight`` ...; the last
 conv_taps - 1 projected rows of a sequence live in its fixed-size state, so such a layer asks
 the cache for keys and values *and* for state); and an output gate sigmoid(W_g x) on the
-concatenated heads (``out_gate``; tensor ``g_proj.weight``, stacked under q | k | v).
+concatenated heads (``out_gate``; tensor ``g_proj.weight``, stacked under q | k | v); biases on
+the q, k and v projections (``qkv_bias``; tensors ``q_proj.bias`` ...); neighbouring dimensions
+rotated as pairs (the position part's ``interleaved``); every value head divided by its root
+mean square before it is cached (``value_norm_eps``); and a soft cap on the scaled scores
+(``softcap``).
 """
 from __future__ import annotations
 
@@ -86,6 +90,15 @@ class AttentionMixer:
         self.conv_taps = int(getattr(spec, "conv_taps", 0) or 0)
         self.out_gate = bool(getattr(spec, "out_gate", False))
         self.conv_w: Optional[torch.Tensor] = None
+        self.softcap = float(getattr(spec, "softcap", None) or 0.0)
+        self.qkv_bias = bool(getattr(spec, "qkv_bias", False))
+        self.bias: Optional[torch.Tensor] = None
+        veps = getattr(spec, "value_norm_eps", None)
+        self.value_eps = None if veps is None else float(veps)
+        self.interleaved = bool(self.position is not None and
+                                getattr(self.position, "interleaved", False))
+        # what only the general norm / rotation / store kernel does
+        self.row_extras = self.qkv_bias or self.interleaved or self.value_eps is not None
         if self.keep_first < 0 or self.conv_taps < 0:
             raise ValueError("keep_first and conv_taps cannot be negative")
         if self.keep_first and self.chunk is not None:
@@ -110,15 +123,18 @@ class AttentionMixer:
                              "rotation, a query temperature or borrowed keys and values")
         if self.fixed_sink is not None and getattr(spec, "sink", False):
             raise ValueError("a sink is either learned or a constant, not both")
-        if self.position is not None and getattr(self.position, "interleaved", False):
-            raise ValueError("this mixer rotates split halves only")
+        if self.row_extras and (self.whole_norm or self.conv_taps or self.out_gate):
+            raise ValueError("biases of the projection, neighbouring pairs and normed values go "
+                             "without a norm over the whole projection, a convolution or an "
+                             "output gate")
         # the options the standard kernels' callers do not pass
         self.plain = (self.own_kv and self.value_dim == spec.head_dim and self.q_temp is None
                       and not getattr(spec, "sink", False) and not self.whole_norm
                       and self.dist_spec is None and self.fixed_sink is None
                       and self.slope_spec is None and self.chunk is None
                       and self.value_mix is None and not self.keep_first
-                      and not self.conv_taps and not self.out_gate)
+                      and not self.conv_taps and not self.out_gate
+                      and not self.row_extras and not self.softcap)
 
     @classmethod
     def param_specs(cls, spec: AttentionSpec, hidden_size: int) -> Dict[str, ParamSpec]:
@@ -153,6 +169,11 @@ class AttentionMixer:
                 p["v_conv.weight"] = ParamSpec((spec.n_kv_heads * vd, taps), "float32")
         if getattr(spec, "out_gate", False):
             p["g_proj.weight"] = ParamSpec((spec.n_heads * vd, hidden_size))
+        if getattr(spec, "qkv_bias", False):
+            p["q_proj.bias"] = ParamSpec((q,), "float32")
+            if own_kv:
+                p["k_proj.bias"] = ParamSpec((kv,), "float32")
+                p["v_proj.bias"] = ParamSpec((spec.n_kv_heads * vd,), "float32")
         return p
 
     @staticmethod
@@ -217,6 +238,10 @@ class AttentionMixer:
             else:
                 self.conv_w = torch.ones((self._conv_channels(), 1), dtype=torch.float32,
                                          device=device)
+        if self.qkv_bias:
+            names = ["q_proj.bias"] + (["k_proj.bias", "v_proj.bias"] if self.own_kv else [])
+            self.bias = torch.cat([tensors[n].to(device=device, dtype=torch.float32)
+                                   for n in names]).contiguous()
         self.out = Linear(mat("o_proj.weight").contiguous(), role="out_proj")
         if self.spec.qk_norm is not None:
             add = 1.0 if self.spec.qk_norm.zero_centered else 0.0
@@ -350,6 +375,7 @@ class AttentionMixer:
         part = proj if proj.dim() == 3 else None
         if (ctx.mode == DECODE and part is not None and hdv == hd and not self.whole_norm and
                 self.dist_bias is None and not self.keep_first and
+                not self.row_extras and not self.softcap and
                 kernels.attention_decode_fused_supported(self.dtype, hd, rotary_dim)):
             out = ctx.new(T, nh * hdv)
             kernels.attention_decode_fused(part, self.q_norm_weight, self.k_norm_weight, eps, cos,
@@ -372,17 +398,19 @@ class AttentionMixer:
         elif self.own_kv:
             if ctx.mode == PREFILL and kernels.attention_prefill_wants_transposed_values(
                     qkv, hd, hdv):
-                vt = kernels.prefill_values_scratch(T, ctx.batch, nkv, hd, qkv.device)
+                vt = kernels.prefill_values_scratch(T, ctx.batch, nkv, hdv, qkv.device)
             kernels.qk_norm_rope_store(
                 qkv, nh, nkv, hd, self.q_norm_weight, self.k_norm_weight, eps, cos, sin,
                 rotary_dim, ctx.positions, view.k_pool, view.v_pool, view.page_table, ctx.slots,
                 ctx.lens, ctx.seq_index, view.page, view.cap, partial=part, vt=vt,
                 cu_seqlens=ctx.cu_seqlens, max_len=ctx.max_new, value_dim=hdv,
-                q_temp=self.q_temp)
+                q_temp=self.q_temp, bias=self.bias, interleaved=self.interleaved,
+                value_eps=self.value_eps)
         else:
             kernels.qk_norm_rope_store(qkv, nh, 0, hd, self.q_norm_weight, None, eps, cos, sin,
                                        rotary_dim, ctx.positions, partial=part, value_dim=hdv,
-                                       q_temp=self.q_temp)
+                                       q_temp=self.q_temp, bias=self.bias,
+                                       interleaved=self.interleaved)
         q = qkv[:, :nh * hd]
         out = ctx.new(T, nh * hdv)
         if ctx.mode == PREFILL:
@@ -394,11 +422,11 @@ class AttentionMixer:
                 k, v, vt = ctx.step_kv[cache_entry]
             kernels.attention_prefill(q, k, v, out, ctx, nh, nkv, hd, s.scale, window, vt=vt,
                                       value_dim=hdv, sinks=self.sinks, dist_bias=self.dist_bias,
-                                      keep_first=self.keep_first)
+                                      keep_first=self.keep_first, softcap=self.softcap)
         else:
             kernels.attention_decode(q, out, view, ctx, nh, nkv, hd, s.scale, window,
                                      value_dim=hdv, sinks=self.sinks, dist_bias=self.dist_bias,
-                                     keep_first=self.keep_first)
+                                     keep_first=self.keep_first, softcap=self.softcap)
         return self.out.partial(out)
 
     def _forward_conv(self, x: torch.Tensor, ctx, cache_entry: int,
@@ -452,11 +480,11 @@ class AttentionMixer:
                 k, v, _ = ctx.step_kv[cache_entry]
             kernels.attention_prefill(q, k, v, out, ctx, nh, nkv, hd, s.scale, window,
                                       value_dim=hdv, sinks=self.sinks, dist_bias=self.dist_bias,
-                                      keep_first=self.keep_first)
+                                      keep_first=self.keep_first, softcap=self.softcap)
         else:
             kernels.attention_decode(q, out, view, ctx, nh, nkv, hd, s.scale, window,
                                      value_dim=hdv, sinks=self.sinks, dist_bias=self.dist_bias,
-                                     keep_first=self.keep_first)
+                                     keep_first=self.keep_first, softcap=self.softcap)
         if self.out_gate:
             kernels.gate_sigmoid(out, qkvg[:, C:])
         return self.out.partial(out)
