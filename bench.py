@@ -348,7 +348,51 @@ def compare_configs_kadavik(size):
     return kadavik, compare_configs_bovozen(size)[0]
 
 
-COMPARE_BUILDERS = {"ramilorn": (compare_configs, "gemma3"),
+# Savovik layer sizes for --compare: width, heads, kv heads, head size, state of the head-wise
+# scan, feed-forward width, layers, vocabulary.
+SAVOVIK_SIZES = {
+    "small": (1024, 16, 4, 64, 64, 4096, 8, 32768),
+    "medium": (2048, 16, 4, 128, 128, 8192, 8, 65536),
+    "large": (4096, 32, 8, 128, 128, 16384, 4, 65536),
+}
+
+
+def compare_configs_savovik(size):
+    """Savovik beside Kadavik, the library's other decoder that sets attention beside a matrix
+    state per head: equal width, heads, head size, layers and vocabulary, dense feed-forwards of
+    equal weight (a gated one has three matrices where the other has two).  Savovik's layers
+    repeat chunked attention beside a selective scan (twice the width, 16 states a channel), the
+    head-wise scan twice (heads of 64, twice the width, one group) and windowed attention with
+    capped scores; Kadavik's alternate attention and the matrix memory."""
+    H, A, G, d, N, ff, L, V = SAVOVIK_SIZES[size]
+    att = {"dim": d, "heads": A, "kv_heads": G, "mask": {"size": 1024},
+           "rot": {"base": 1000000.0, "dims": d, "scaling": {"factor": 4.0}},
+           "scale": d ** -0.5, "softcap": 50.0, "vdim": d}
+    left = {"dim": d, "heads": A, "kv_heads": G, "mask": {"size": 1024},
+            "rot": {"base": 1000000.0, "dims": d // 2,
+                    "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}},
+            "scale": d ** -0.5, "vdim": d}
+    par = {"left": left, "left_scale": 1.2, "right_scale": 0.8,
+           "right": {"conv": 4, "dt_rank": H // 16, "inner": 2 * H, "state": 16}}
+    ssm = {"conv": 4, "groups": 1, "heads": 2 * H // 64, "norm_groups": 1, "state": N, "vdim": 64}
+    kinds = [("parallel", par), ("mamba2", ssm), ("mamba2", ssm), ("attention", att)]
+    layers = [{"mixer": kinds[l % 4][1], "mlp": {"ff": ff, "kind": "dense"}, "type": kinds[l % 4][0]}
+              for l in range(L)]
+    savovik = {"architecture": "Savovik", "layers": layers, "norm": {"eps": 1e-6}, "vocab": V,
+               "width": H}
+    katt = {"conv": 4, "dim": d, "heads": A, "kv_heads": G, "mask": {"keep_first": 0, "size": 1024},
+            "rot": {"base": 1000000.0, "dims": d // 2}, "scale": d ** -0.5, "vdim": d}
+    rec = {"dim": d, "gate_cap": 15.0, "heads": A, "vdim": d}
+    mlp = {"ff": ff * 2 // 3 // 128 * 128, "kind": "dense"}
+    klayers = [{"mixer": rec if l % 2 else katt, "mlp": mlp,
+                "type": "mlstm" if l % 2 else "attention"} for l in range(L)]
+    kadavik = {"architecture": "Kadavik", "embedding": {"scale": H ** 0.5}, "layers": klayers,
+               "logit_scale": 1.0, "norm": {"eps": 1e-6}, "vocab": V, "width": H}
+    return savovik, kadavik
+
+
+COMPARE_BUILDERS = {"savovik": (compare_configs_savovik, "kadavik"),
+                    "ramilorn": (compare_configs, "gemma3"),
                     "kadavik": (compare_configs_kadavik, "bovozen"),
                     "zazerax": (compare_configs_zazerax, "gemma3"),
                     "bovozen": (compare_configs_bovozen, "ramilorn")}
