@@ -116,8 +116,9 @@ __device__ __forceinline__ float distance_bias(const DecodeArgs& a, int p, int j
 }
 
 // The scaled score under the soft cap, if there is one.
+template <bool EXT>
 __device__ __forceinline__ float capped(const DecodeArgs& a, float s) {
-    return a.softcap > 0.f ? soft_capped_ex2(s, 2.0f * 1.4426950408889634f / a.softcap, a.softcap) : s;
+    return EXT && a.softcap > 0.f ? soft_capped_ex2(s, 2.0f * 1.4426950408889634f / a.softcap, a.softcap) : s;
 }
 
 // What the sink of head h adds to a normaliser taken relative to the maximum m.
@@ -156,11 +157,11 @@ struct FuseQK {
 template <typename T>
 __device__ __forceinline__ void finish_split(const DecodeArgs& a, int b, int h0, int gc, int used,
                                              int split, float* stat, float* wts, int wcap,
-                                             int* s_last, T* outp, int arrivals = 0,
+                                             int* s_last, T* outp, int hdv, int arrivals = 0,
                                              bool write_ml = true) {
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int nthreads = blockDim.x, nwarps = nthreads >> 5;
-    const int hd = a.hdv;                      // (values only from here on)
+    const int hd = hdv;                        // (values only from here on)
     if (arrivals == 0) arrivals = used;        // one arrival per partial result
     if (write_ml && tid < gc) {
         float* dst = a.part_ml + (((size_t)b * a.nh + h0 + tid) * a.n_splits + split) * 2;
@@ -390,7 +391,7 @@ attention_decode_split_kernel(DecodeArgs a) {
     }
     if (used == 1) return;
     finish_split<T>(a, b, h0, gc, used, split, stat, reinterpret_cast<float*>(smem_raw),
-                    (int)(((size_t)CH * (hd + hdv) * sizeof(T)) / sizeof(float)), &s_last, outp);
+                    (int)(((size_t)CH * (hd + hdv) * sizeof(T)) / sizeof(float)), &s_last, outp, hdv);
 }
 
 // ------------------------------------------------------- tensor-core variant
@@ -587,7 +588,9 @@ struct PoolMaps {
 template <>
 struct PoolMaps<false> {};
 
-template <int HDP, bool TMA>
+// EXT: the form with a soft cap and value heads of their own size (a form of its own, so that
+// the plain form, a decode step's longest chain, keeps its registers and its instructions).
+template <int HDP, bool TMA, bool EXT>
 __global__ void __launch_bounds__(DmShape<HDP>::NT, DmShape<HDP>::NT == 256 ? 2 : 3)
 attention_decode_mma_kernel(DecodeArgs a, int cs, FuseQK fq,
                             const __grid_constant__ PoolMaps<TMA> maps) {
@@ -630,7 +633,7 @@ attention_decode_mma_kernel(DecodeArgs a, int cs, FuseQK fq,
     const int g = blockIdx.y / groups_per_kv;
     const int h0 = g * G + (blockIdx.y % groups_per_kv) * DM_HEADS;
     const int gc = min(DM_HEADS, g * G + G - h0);
-    const int hd = a.hd, hdv = a.hdv;
+    const int hd = a.hd, hdv = EXT ? a.hdv : a.hd;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int gid = lane >> 2, tig = lane & 3;
     T* outp = (T*)a.out + ((size_t)b * a.nh + h0) * hdv;
@@ -770,6 +773,17 @@ attention_decode_mma_kernel(DecodeArgs a, int cs, FuseQK fq,
             const int r = i / CPR, c = i % CPR;
             const int off = dm_swz<HDP>(r, c);
             if (r == skip) continue;
+            if (!EXT) {
+                if (ro[r] >= 0 && c * 8 < hd) {
+                    const size_t src = ((size_t)ro[r] * a.nkv + g) * hd + c * 8;
+                    cp_async16(kd + off, (const T*)a.k_pool + src);
+                    cp_async16(vd + off, (const T*)a.v_pool + src);
+                } else {
+                    *reinterpret_cast<uint4*>(kd + off) = make_uint4(0, 0, 0, 0);
+                    *reinterpret_cast<uint4*>(vd + off) = make_uint4(0, 0, 0, 0);
+                }
+                continue;
+            }
             const size_t head = (size_t)ro[r] * a.nkv + g;
             if (ro[r] >= 0 && c * 8 < hd)
                 cp_async16(kd + off, (const T*)a.k_pool + head * hd + c * 8);
@@ -857,6 +871,17 @@ attention_decode_mma_kernel(DecodeArgs a, int cs, FuseQK fq,
         }
         for (int c = tid; c < CPR; c += DM_THREADS) {
             const int off = kv_swz<HDP, TMA>(r, c);
+            if (!EXT) {
+                if (cache_row >= 0 && c * 8 < hd) {
+                    const size_t src = ((size_t)cache_row * a.nkv + g) * hd + c * 8;
+                    cp_async16(Ks + off, (const T*)a.k_pool + src);
+                    cp_async16(Vs + off, (const T*)a.v_pool + src);
+                } else {
+                    *reinterpret_cast<uint4*>(Ks + off) = make_uint4(0, 0, 0, 0);
+                    *reinterpret_cast<uint4*>(Vs + off) = make_uint4(0, 0, 0, 0);
+                }
+                continue;
+            }
             const size_t head = (size_t)cache_row * a.nkv + g;
             if (cache_row >= 0 && c * 8 < hd)
                 cp_async16(Ks + off, (const T*)a.k_pool + head * hd + c * 8);
@@ -960,7 +985,7 @@ attention_decode_mma_kernel(DecodeArgs a, int cs, FuseQK fq,
             for (int e = 0; e < 4; ++e) {
                 const int key = warp * 16 + i * 8 + tig * 2 + (e & 1);
                 const int row = gid + (e >> 1) * 8;
-                float sv = key >= nlo && key < n ? capped(a, s[i][e] * a.scale) : -INFINITY;
+                float sv = key >= nlo && key < n ? capped<EXT>(a, s[i][e] * a.scale) : -INFINITY;
                 // (with a distance bias the tiles come by copies, so jt + key is the position)
                 if (!TMA && a.dist_bias && row < gc && key >= nlo && key < n)
                     sv += distance_bias(a, p, jt + key, h0 + row);
@@ -986,7 +1011,7 @@ attention_decode_mma_kernel(DecodeArgs a, int cs, FuseQK fq,
             const int key = warp * 8 + tig * 2 + (e & 1);
             const int row = gid + (e >> 1) * 8;
             float sv = key >= nlo && key < n
-                ? capped(a, ((s[0][e] + s[1][e]) + (s[2][e] + s[3][e])) * a.scale) : -INFINITY;
+                ? capped<EXT>(a, ((s[0][e] + s[1][e]) + (s[2][e] + s[3][e])) * a.scale) : -INFINITY;
             if (!TMA && a.dist_bias && row < gc && key >= nlo && key < n)
                 sv += distance_bias(a, p, jt + key, h0 + row);
             Ss[row * DM_KEYS + key] = sv;
@@ -1098,7 +1123,7 @@ attention_decode_mma_kernel(DecodeArgs a, int cs, FuseQK fq,
     const int wcap = (int)((size_t)2 * DM_KEYS * HDP * sizeof(T) / sizeof(float));
     if (cs == 1) {
         finish_split<T>(a, b, h0, gc, used, split, stat, reinterpret_cast<float*>(smem_raw), wcap,
-                        &s_last, outp);
+                        &s_last, outp, hdv);
         return;
     }
     // ---- merge inside the cluster: rank r owns a slice of the head dimension
@@ -1146,7 +1171,7 @@ attention_decode_mma_kernel(DecodeArgs a, int cs, FuseQK fq,
     if (used_clusters == 1) return;
     // a long sequence: one partial result per cluster, merged by the last CTA to arrive
     finish_split<T>(a, b, h0, gc, used_clusters, cid, stat, reinterpret_cast<float*>(smem_raw), wcap,
-                    &s_last, outp, used_clusters * cs, false);
+                    &s_last, outp, hdv, used_clusters * cs, false);
 }
 
 // A pool [rows, nkv, hd] bfloat16 as a 3-D tensor map read in boxes of [64 rows, 1 head, 64
@@ -1228,9 +1253,9 @@ int most_tiles(const DecodeArgs& a, bool pages) {
     return a.n_splits + (pages && a.window != 0 && a.cap != a.window ? 1 : 0);
 }
 
-template <int HDP, bool TMA>
+template <int HDP, bool TMA, bool EXT>
 int launch_decode_mma(const DecodeArgs& a0, int B, cudaStream_t stream, const FuseQK& fq) {
-    auto kern = attention_decode_mma_kernel<HDP, TMA>;
+    auto kern = attention_decode_mma_kernel<HDP, TMA, EXT>;
     constexpr int DM_THREADS = DmShape<HDP>::NT;
     constexpr int NBUF = TMA ? DmShape<HDP>::NBUF_TMA : DmShape<HDP>::NBUF;
     constexpr int smem = (2 * NBUF * DM_KEYS + DM_HEADS) * HDP * 2 + DM_HEADS * DM_KEYS * (2 + 4) +
@@ -1296,8 +1321,12 @@ int launch_decode_form(const DecodeArgs& a, int B, cudaStream_t stream, const Fu
         const bool ring = a.window > 0 && a.cap == a.window;
         tma = most >= (ring ? 2 : DmShape<HDP>::NBUF_TMA == 3 ? 4 : 6) * cs * clusters;
     }
-    if (tma) return launch_decode_mma<HDP, true>(a, B, stream, fq);
-    return launch_decode_mma<HDP, false>(a, B, stream, fq);
+    const bool ext = a.softcap > 0.f || a.hdv != a.hd;
+    if (tma)
+        return ext ? launch_decode_mma<HDP, true, true>(a, B, stream, fq)
+                   : launch_decode_mma<HDP, true, false>(a, B, stream, fq);
+    return ext ? launch_decode_mma<HDP, false, true>(a, B, stream, fq)
+               : launch_decode_mma<HDP, false, false>(a, B, stream, fq);
 }
 
 int pick_chunk(int hd, int elem) {                  // hd: the wider of a key and a value head

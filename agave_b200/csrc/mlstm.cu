@@ -92,6 +92,7 @@ template <int N> __device__ __forceinline__ void cp_async_wait() {
 // what another writes.
 //
 // NORM false: there is no last warp and no n or m; the factors a_t, b_t come with the tokens.
+// CPT: columns a lane holds, 32 apart (a piece of k or q read once serves them all).
 struct ScanIn {
     const float *q, *k, *v;    // the first token's; a head's q and k start (h / shared) * d behind
     long long ld;              // between tokens
@@ -99,7 +100,7 @@ struct ScanIn {
     const float* gates;        // NORM: [T, 2 H] log gates (i, then f); else [T, H, 2] (a, b)
 };
 
-template <int RW, bool NORM>
+template <int RW, bool NORM, int CPT>
 __global__ void __launch_bounds__((RW + (NORM ? 1 : 0)) * 32)
 mlstm_scan_kernel(ScanIn in, float* __restrict__ num, float* __restrict__ den, int H, int d, int dv,
                   float* __restrict__ state, long long state_stride, long long state_off,
@@ -111,7 +112,8 @@ mlstm_scan_kernel(ScanIn in, float* __restrict__ num, float* __restrict__ den, i
     constexpr int NR = RW >= 2 ? RW / 2 : 1;          // rows of n a lane of the last warp holds
     constexpr int CH = ML_CHUNK;
     static_assert(2 * CH <= 32, "a warp copies the factors of a chunk");
-    constexpr int CW = ML_COLS;
+    constexpr int CW = ML_COLS * CPT;
+    static_assert(!NORM || CPT == 1, "the form with a normaliser holds one column a lane");
     constexpr int BUF = CH * (2 * DP + CW);
     constexpr int NWARPS = RW + (NORM ? 1 : 0);
     const float* __restrict__ gates = in.gates;
@@ -122,13 +124,17 @@ mlstm_scan_kernel(ScanIn in, float* __restrict__ num, float* __restrict__ den, i
     const int slot = slots[b];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const bool is_nw = NORM && warp == RW;
-    const int col = blockIdx.x * CW + lane;
-    const bool live = col < dv;
+    const int col = blockIdx.x * CW + lane;           // and CPT - 1 more, 32 apart
+    bool live[CPT];
+#pragma unroll
+    for (int x = 0; x < CPT; ++x) live[x] = col + 32 * x < dv;
     const int hg = h / in.shared;
     if (slot < 0) {
         // a padding entry: its rows are written, with zeros
         for (int t = t0; t < t1; ++t) {
-            if (warp == 0 && live) num[(size_t)t * H * dv + (size_t)h * dv + col] = 0.f;
+#pragma unroll
+            for (int x = 0; x < CPT; ++x)
+                if (warp == 0 && live[x]) num[(size_t)t * H * dv + (size_t)h * dv + col + 32 * x] = 0.f;
             if (is_nw && lane == 0 && blockIdx.x == 0) {
                 den[((size_t)t * H + h) * 2] = 0.f;
                 den[((size_t)t * H + h) * 2 + 1] = 1.f;
@@ -141,20 +147,21 @@ mlstm_scan_kernel(ScanIn in, float* __restrict__ num, float* __restrict__ den, i
     float* n_g = st + (size_t)H * d * dv + (size_t)h * d;
     float* m_g = st + (size_t)H * d * dv + (size_t)H * d + (size_t)h * mlstm_m_copies(dv) +
                  (blockIdx.x * CW) / ML_MCOLS;
-    // a row warp's thread: S[j] = row warp * 16 + j of its column; the last warp's: its rows
-    // j * 32 + lane of n in S[0 .. NR)
-    float S[ML_ROWS];
+    // a row warp's thread: S[j] = rows warp * 16 + 2 j and + 1 of its column; the last warp's:
+    // its rows j * 32 + lane of n
+    f32x2 S[CPT][ML_ROWS / 2];                        // two rows each
+    float nrow[NR];
 #pragma unroll
-    for (int j = 0; j < ML_ROWS; ++j) {
-        S[j] = 0.f;
-        if (!is_nw) {
-            const int r = warp * ML_ROWS + j;
-            if (live && r < d) S[j] = S_g[(size_t)r * dv + col];
-        } else if (j < NR) {
-            const int r = j * 32 + lane;
-            if (r < d) S[j] = n_g[r];
+    for (int x = 0; x < CPT; ++x)
+#pragma unroll
+        for (int j = 0; j < ML_ROWS / 2; ++j) {
+            const int r = warp * ML_ROWS + 2 * j;
+            const float* at = S_g + (size_t)r * dv + col + 32 * x;
+            const bool mine = !is_nw && live[x];
+            S[x][j] = pack2(mine && r < d ? at[0] : 0.f, mine && r + 1 < d ? at[dv] : 0.f);
         }
-    }
+#pragma unroll
+    for (int j = 0; j < NR; ++j) nrow[j] = is_nw && j * 32 + lane < d ? n_g[j * 32 + lane] : 0.f;
     // the padding rows of both buffers stay zero
     for (int i = threadIdx.x; i < 2 * BUF; i += blockDim.x) sm[i] = 0.f;
     __syncthreads();
@@ -173,7 +180,10 @@ mlstm_scan_kernel(ScanIn in, float* __restrict__ num, float* __restrict__ den, i
                 cp_async4(qs + tt * DP + r, qr + r);
                 cp_async4(ks + tt * DP + r, kr + r);
             }
-            if (live) cp_async4(vs + tt * CW + lane, in.v + at + (size_t)h * dv + col);
+#pragma unroll
+            for (int x = 0; x < CPT; ++x)
+                if (live[x])
+                    cp_async4(vs + tt * CW + lane + 32 * x, in.v + at + (size_t)h * dv + col + 32 * x);
         }
         if (!NORM && warp == 0 && lane < 2 * nt)
             cp_async4(coef + (c & 1) * CH * 2 + lane,
@@ -240,28 +250,40 @@ mlstm_scan_kernel(ScanIn in, float* __restrict__ num, float* __restrict__ den, i
         const float* ks = qs + CH * DP;
         const float* vs = ks + CH * DP;
         if (!is_nw) {
-            const float4* kbase = reinterpret_cast<const float4*>(ks + warp * ML_ROWS);
-            const float4* qbase = reinterpret_cast<const float4*>(qs + warp * ML_ROWS);
+            const ulonglong2* kbase = reinterpret_cast<const ulonglong2*>(ks + warp * ML_ROWS);
+            const ulonglong2* qbase = reinterpret_cast<const ulonglong2*>(qs + warp * ML_ROWS);
 #pragma unroll 2
             for (int tt = 0; tt < nt; ++tt) {
                 const float a = cf[tt * 2];
-                const float wv = cf[tt * 2 + 1] * vs[tt * CW + lane];
-                const float4* k4 = kbase + tt * (DP / 4);
-                const float4* q4 = qbase + tt * (DP / 4);
-                float acc[4] = {0.f, 0.f, 0.f, 0.f};
+                f32x2 wv[CPT], acc[CPT][2];
+                const f32x2 aa = pack2(a, a);
+#pragma unroll
+                for (int x = 0; x < CPT; ++x) {
+                    const float w = cf[tt * 2 + 1] * vs[tt * CW + lane + 32 * x];
+                    wv[x] = pack2(w, w);
+                    acc[x][0] = acc[x][1] = 0;
+                }
+                const ulonglong2* k4 = kbase + tt * (DP / 4);
+                const ulonglong2* q4 = qbase + tt * (DP / 4);
 #pragma unroll
                 for (int j = 0; j < ML_ROWS / 4; ++j) {
-                    const float4 kk = k4[j], qq = q4[j];
-                    S[j * 4 + 0] = fmaf(wv, kk.x, a * S[j * 4 + 0]);
-                    S[j * 4 + 1] = fmaf(wv, kk.y, a * S[j * 4 + 1]);
-                    S[j * 4 + 2] = fmaf(wv, kk.z, a * S[j * 4 + 2]);
-                    S[j * 4 + 3] = fmaf(wv, kk.w, a * S[j * 4 + 3]);
-                    acc[0] = fmaf(S[j * 4 + 0], qq.x, acc[0]);
-                    acc[1] = fmaf(S[j * 4 + 1], qq.y, acc[1]);
-                    acc[2] = fmaf(S[j * 4 + 2], qq.z, acc[2]);
-                    acc[3] = fmaf(S[j * 4 + 3], qq.w, acc[3]);
+                    const ulonglong2 kk = k4[j], qq = q4[j];
+#pragma unroll
+                    for (int x = 0; x < CPT; ++x) {
+                        f32x2* s = S[x] + j * 2;
+                        s[0] = fma2(wv[x], kk.x, mul2(aa, s[0]));
+                        s[1] = fma2(wv[x], kk.y, mul2(aa, s[1]));
+                        acc[x][0] = fma2(s[0], qq.x, acc[x][0]);
+                        acc[x][1] = fma2(s[1], qq.y, acc[x][1]);
+                    }
                 }
-                ps[(tt * RW + warp) * CW + lane] = (acc[0] + acc[1]) + (acc[2] + acc[3]);
+#pragma unroll
+                for (int x = 0; x < CPT; ++x) {
+                    float p0, p1, p2, p3;
+                    unpack2(acc[x][0], p0, p1);
+                    unpack2(acc[x][1], p2, p3);
+                    ps[(tt * RW + warp) * CW + lane + 32 * x] = (p0 + p1) + (p2 + p3);
+                }
             }
         } else {
             // n over the chunk, each lane's part of every token's n . q kept; then the warp
@@ -277,8 +299,8 @@ mlstm_scan_kernel(ScanIn in, float* __restrict__ num, float* __restrict__ den, i
                         const int r = j * 32 + lane;
                         const float kk = r < DP ? ks[tt * DP + r] : 0.f;
                         const float qq = r < DP ? qs[tt * DP + r] : 0.f;
-                        S[j] = fmaf(w, kk, a * S[j]);
-                        dn[tt] = fmaf(S[j], qq, dn[tt]);
+                        nrow[j] = fmaf(w, kk, a * nrow[j]);
+                        dn[tt] = fmaf(nrow[j], qq, dn[tt]);
                     }
                 }
             }
@@ -306,15 +328,22 @@ mlstm_scan_kernel(ScanIn in, float* __restrict__ num, float* __restrict__ den, i
         }
     }
     if (t1 > t0) {
+        if (!is_nw) {
 #pragma unroll
-        for (int j = 0; j < ML_ROWS; ++j) {
-            if (!is_nw) {
-                const int r = warp * ML_ROWS + j;
-                if (live && r < d) S_g[(size_t)r * dv + col] = S[j];
-            } else if (j < NR && blockIdx.x == 0) {
-                const int r = j * 32 + lane;
-                if (r < d) n_g[r] = S[j];
-            }
+            for (int x = 0; x < CPT; ++x)
+#pragma unroll
+                for (int j = 0; j < ML_ROWS / 2; ++j) {
+                    const int r = warp * ML_ROWS + 2 * j;
+                    float* at = S_g + (size_t)r * dv + col + 32 * x;
+                    float lo, hi;
+                    unpack2(S[x][j], lo, hi);
+                    if (live[x] && r < d) at[0] = lo;
+                    if (live[x] && r + 1 < d) at[dv] = hi;
+                }
+        } else if (blockIdx.x == 0) {
+#pragma unroll
+            for (int j = 0; j < NR; ++j)
+                if (j * 32 + lane < d) n_g[j * 32 + lane] = nrow[j];
         }
         if (is_nw && lane == 0) {
             const int mine = min(CW, dv - (int)blockIdx.x * CW);
@@ -362,18 +391,19 @@ int row_in(RowIn<float>& in, const float* row, long long ld, const float* part, 
     return 0;
 }
 
-template <bool NORM>
+template <bool NORM, int CPT>
 int launch_scan(const ScanIn& in, float* num, float* den, int B, int H, int d, int dv, float* state,
                 long long state_stride, long long state_off, const int* slots,
                 const int* cu_seqlens, cudaStream_t stream) {
     int RW = 1;
     while (RW * ML_ROWS < d) RW *= 2;
-    const dim3 grid((unsigned)((dv + ML_COLS - 1) / ML_COLS), (unsigned)H, (unsigned)B);
-    const size_t smem = ((size_t)2 * ML_CHUNK * (2 * RW * ML_ROWS + ML_COLS) + 4 * ML_CHUNK +
-                         (size_t)2 * ML_CHUNK * RW * ML_COLS) * sizeof(float);
+    constexpr int CW = ML_COLS * CPT;
+    const dim3 grid((unsigned)((dv + CW - 1) / CW), (unsigned)H, (unsigned)B);
+    const size_t smem = ((size_t)2 * ML_CHUNK * (2 * RW * ML_ROWS + CW) + 4 * ML_CHUNK +
+                         (size_t)2 * ML_CHUNK * RW * CW) * sizeof(float);
 #define AGV_SCAN(RR)                                                                          \
     do {                                                                                      \
-        auto kern = mlstm_scan_kernel<RR, NORM>;                                              \
+        auto kern = mlstm_scan_kernel<RR, NORM, CPT>;                                              \
         static bool configured = false;          /* (the size follows from RR alone) */       \
         if (smem > 48 * 1024 && !configured) {                                                \
             AGV_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, \
@@ -428,7 +458,7 @@ AGV_API int agv_mlstm_scan(const float* qkv, const float* gates, float* num, flo
     if (T == 0) return 0;
     const ScanIn in{qkv, qkv + (size_t)H * d, qkv + (size_t)2 * H * d, 2LL * H * d + (long long)H * dv,
                     1, gates};
-    return launch_scan<true>(in, num, den, B, H, d, dv, state, state_stride, 0, slots, cu_seqlens,
+    return launch_scan<true, 1>(in, num, den, B, H, d, dv, state, state_stride, 0, slots, cu_seqlens,
                              stream);
 }
 
@@ -446,8 +476,16 @@ AGV_API int agv_head_scan(const float* q, const float* k, const float* v, long l
     AGV_REQUIRE(B <= 65535 && H <= 65535, "head_scan: batch or head count exceeds the grid limit");
     if (T == 0) return 0;
     const ScanIn in{q, k, v, ld, H / groups, coef};
-    return launch_scan<false>(in, out, nullptr, B, H, d, dv, state, state_stride, state_off, slots,
-                              cu_seqlens, stream);
+    // Two columns a lane halve the reads of k and q but also the warps that hide a token's
+    // latencies: taken where one column a lane would put a second CTA on most SMs anyway (2,048
+    // tokens, 128 heads of 128 x 64: 475 us against 555; 64 such heads: 475 against 367), and
+    // not while decoding, where a token is a read and a write of the state.
+    const long long ctas = (long long)((dv + ML_COLS - 1) / ML_COLS) * H * B;
+    if (dv > ML_COLS && ctas > 192 && T > B)
+        return launch_scan<false, 2>(in, out, nullptr, B, H, d, dv, state, state_stride, state_off,
+                                     slots, cu_seqlens, stream);
+    return launch_scan<false, 1>(in, out, nullptr, B, H, d, dv, state, state_stride, state_off, slots,
+                                 cu_seqlens, stream);
 }
 
 AGV_API int agv_mlstm_out(const float* num, const float* den, float den_eps, const float* row,

@@ -22,6 +22,12 @@ struct RowIn {
         }
         return to_f32(row[(size_t)t * ld + e]);
     }
+    // The 32-bit rows themselves, where there is one sum a value, and their stride; else null.
+    __device__ __forceinline__ const float* single(long long& stride) const {
+        stride = part ? W : ld;
+        if (part) return n_splits == 1 ? part : nullptr;
+        return sizeof(T) == sizeof(float) ? reinterpret_cast<const float*>(row) : nullptr;
+    }
     // The whole row of token t into shared memory, 32-bit: eight values per thread at a
     // time with all their loads issued before the first is used (a dependent trip to L2 or
     // HBM costs about a microsecond, and a decode step has few rows to hide it behind).

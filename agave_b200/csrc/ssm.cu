@@ -57,8 +57,19 @@ ssm_conv_kernel(RowIn<float> in, int n_tokens, int off, int C, StepArgs st,
     pdl_wait();
     pdl_launch_next();
     constexpr int RING = TAPS - 1, MOD = RING > 0 ? RING : 1;
+    // what the tile's tokens are: position, tokens of the sequence in this step before it, slot,
+    // and whether the token is among the sequence's last inputs
+    __shared__ int s_pos[R], s_in[R], s_slot[R], s_keep[R];
     const int c = blockIdx.x * 128 + threadIdx.x;
     const int t0 = blockIdx.y * R;
+    if (threadIdx.x < R && t0 + threadIdx.x < n_tokens) {
+        const int t = t0 + threadIdx.x, e = st.seq_index[t], p = st.positions[t];
+        s_pos[threadIdx.x] = p;
+        s_in[threadIdx.x] = t - st.cu[e];
+        s_slot[threadIdx.x] = st.slots[e];
+        s_keep[threadIdx.x] = p >= st.lens[e] - RING;
+    }
+    __syncthreads();
     if (c >= C + n_dt) return;
     if (c >= C) {
         const int h = c - C;
@@ -77,24 +88,32 @@ ssm_conv_kernel(RowIn<float> in, int n_tokens, int off, int C, StepArgs st,
 #pragma unroll
     for (int j = 0; j < TAPS; ++j) wv[j] = w[(size_t)c * TAPS + j];
     const float b = bias[c];
+    long long ld;
+    if (const float* src = in.single(ld)) {                    // (all loads in flight at once)
 #pragma unroll
-    for (int i = 0; i < R + RING; ++i) {
-        const int t = t0 - RING + i;
-        xs[i] = t >= 0 && t < n_tokens ? in.at(t, off + c) : 0.f;
+        for (int i = 0; i < R + RING; ++i) {
+            const int t = t0 - RING + i;
+            xs[i] = t >= 0 && t < n_tokens ? src[(size_t)t * ld + off + c] : 0.f;
+        }
+    } else {
+#pragma unroll
+        for (int i = 0; i < R + RING; ++i) {
+            const int t = t0 - RING + i;
+            xs[i] = t >= 0 && t < n_tokens ? in.at(t, off + c) : 0.f;
+        }
     }
 #pragma unroll
     for (int i = 0; i < R; ++i) {
         const int t = t0 + i;
         if (t >= n_tokens) break;
-        const int e = st.seq_index[t], slot = st.slots[e], p = st.positions[t];
-        const int first = st.cu[e];
+        const int p = s_pos[i], slot = s_slot[i], before = s_in[i];
         float* ring = slot >= 0 && RING > 0 ? st.state + (size_t)slot * st.stride + st.off + c : nullptr;
         float acc = b;
 #pragma unroll
         for (int k = RING; k >= 1; --k) {                      // oldest input first
             float x = 0.f;
             if (p - k >= 0) {
-                if (t - k >= first) x = xs[RING + i - k];
+                if (k <= before) x = xs[RING + i - k];
                 else if (ring) x = ring[(size_t)((p - k) % MOD) * C];
             }
             acc = fmaf(wv[RING - k], x, acc);
@@ -103,7 +122,7 @@ ssm_conv_kernel(RowIn<float> in, int n_tokens, int off, int C, StepArgs st,
         const float y = silu_f(fmaf(wv[RING], cur, acc));
         out[(size_t)t * C + c] = y;
         if (rounded) rounded[(size_t)t * C + c] = from_f32<T>(y);
-        if (ring && p >= st.lens[e] - RING) ring[(size_t)(p % MOD) * C] = cur;
+        if (ring && s_keep[i]) ring[(size_t)(p % MOD) * C] = cur;
     }
 }
 
@@ -162,7 +181,7 @@ selective_scan_kernel(SelectiveArgs a, RowIn<float> in, StepArgs st, T* __restri
     pdl_wait();
     extern __shared__ __align__(16) float sm[];
     constexpr int CC = SS_THREADS / L, Np = NS * L, CH = SS_CH;
-    constexpr int BUF = CH * (2 * CC + 2 * Np);
+    constexpr int BUF = CH * (3 * CC + 2 * Np);
     constexpr int ZN = CH * CC / SS_THREADS > 0 ? CH * CC / SS_THREADS : 1;
     float2* dd = reinterpret_cast<float2*>(sm + 2 * BUF);     // [CH][CC] (dt, dt u)
     float* ys = reinterpret_cast<float*>(dd + CH * CC);       // [CH][CC]
@@ -179,11 +198,16 @@ selective_scan_kernel(SelectiveArgs a, RowIn<float> in, StepArgs st, T* __restri
     }
     for (int i = tid; i < 2 * BUF; i += SS_THREADS) sm[i] = 0.f;   // (what is never copied stays zero)
     __syncthreads();
-    const bool vec = a.inner % 4 == 0 && CC % 4 == 0;
+    // z comes with the tokens where it is one sum, else its partial sums are added up below
+    long long zld;
+    const float* zrow = in.single(zld);
+    if (zrow) zrow += a.z_off;
+    const bool vec = a.inner % 4 == 0 && CC % 4 == 0 &&
+                     (!zrow || (zld % 4 == 0 && ((uintptr_t)zrow & 15) == 0));
     auto fetch = [&](int ch) {
         float* base = sm + (ch & 1) * BUF;
         const int c0 = ch * CH, m = min(CH, n - c0);
-        float *ds = base, *us = ds + CH * CC, *bs = us + CH * CC;
+        float *ds = base, *us = ds + CH * CC, *zs = us + CH * CC, *bs = zs + CH * CC;
         if (vec) {
             constexpr int Q = CC / 4 > 0 ? CC / 4 : 1;
             for (int i = tid; i < m * Q; i += SS_THREADS) {
@@ -192,6 +216,7 @@ selective_scan_kernel(SelectiveArgs a, RowIn<float> in, StepArgs st, T* __restri
                     const size_t src = (size_t)(t0 + c0 + tt) * a.inner + cb + k;
                     cp_async_16(ds + tt * CC + k, a.dt + src);
                     cp_async_16(us + tt * CC + k, a.u + src);
+                    if (zrow) cp_async_16(zs + tt * CC + k, zrow + (size_t)(t0 + c0 + tt) * zld + cb + k);
                 }
             }
         } else {
@@ -201,6 +226,7 @@ selective_scan_kernel(SelectiveArgs a, RowIn<float> in, StepArgs st, T* __restri
                     const size_t src = (size_t)(t0 + c0 + tt) * a.inner + cb + k;
                     cp_async_4(ds + i, a.dt + src);
                     cp_async_4(us + i, a.u + src);
+                    if (zrow) cp_async_4(zs + i, zrow + (size_t)(t0 + c0 + tt) * zld + cb + k);
                 }
             }
         }
@@ -218,27 +244,24 @@ selective_scan_kernel(SelectiveArgs a, RowIn<float> in, StepArgs st, T* __restri
         S[s] = ok ? srow[k] : 0.f;
         a2[s] = ok ? a.a2[(size_t)c * a.N + k] : 0.f;
     }
+    // outside the recurrence a thread's places of a chunk all have one channel
+    const int my_c = cb + tid % CC;
+    const bool mine = my_c < a.inner;
+    const float my_bias = mine ? a.dt_bias[my_c] : 0.f, my_d = mine ? a.D[my_c] : 0.f;
     const int n_chunks = (n + CH - 1) / CH;
     for (int ch = 0; ch < n_chunks; ++ch) {
         const int c0 = ch * CH, m = min(CH, n - c0);
         const float* base = sm + (ch & 1) * BUF;
-        const float *ds = base, *us = ds + CH * CC, *bs = us + CH * CC;
-        // the gate's values of this chunk's outputs are on their way while it runs
-        float z[ZN];
-#pragma unroll
-        for (int i = 0; i < ZN; ++i) {
-            const int k = tid + i * SS_THREADS, tt = k / CC, cc = cb + k % CC;
-            z[i] = tt < m && cc < a.inner ? in.at(t0 + c0 + tt, a.z_off + cc) : 0.f;
-        }
+        const float *ds = base, *us = ds + CH * CC, *zs = us + CH * CC, *bs = zs + CH * CC;
         cp_async_wait<0>();
         __syncthreads();
         if (ch + 1 < n_chunks) fetch(ch + 1);
 #pragma unroll
         for (int i = 0; i < ZN; ++i) {
-            const int k = tid + i * SS_THREADS, tt = k / CC, cc = cb + k % CC;
+            const int k = tid + i * SS_THREADS, tt = k / CC;
             float2 v = make_float2(0.f, 0.f);
-            if (k < CH * CC && tt < m && cc < a.inner) {
-                v.x = softplus_f(ds[k] + a.dt_bias[cc]);
+            if (k < CH * CC && tt < m && mine) {
+                v.x = softplus_f(ds[k] + my_bias);
                 v.y = v.x * us[k];
             }
             if (k < CH * CC) dd[k] = v;
@@ -249,8 +272,8 @@ selective_scan_kernel(SelectiveArgs a, RowIn<float> in, StepArgs st, T* __restri
 #pragma unroll
             for (int q = 0; q < 4; ++q) {
                 const float2 d = dd[(tt + q) * CC + jc];
-                float B[NS], Cv[NS];
                 const float* row = bs + (tt + q) * 2 * Np + l * NS;
+                float B[NS], Cv[NS];
                 if constexpr (NS % 4 == 0) {
 #pragma unroll
                     for (int s = 0; s < NS; s += 4) {
@@ -297,10 +320,11 @@ selective_scan_kernel(SelectiveArgs a, RowIn<float> in, StepArgs st, T* __restri
         __syncthreads();
 #pragma unroll
         for (int i = 0; i < ZN; ++i) {
-            const int k = tid + i * SS_THREADS, tt = k / CC, cc = cb + k % CC;
-            if (tt < m && cc < a.inner) {
-                const float y = fmaf(a.D[cc], us[k], ys[k]);
-                out[(size_t)(t0 + c0 + tt) * a.inner + cc] = from_f32<T>(y * silu_f(z[i]));
+            const int k = tid + i * SS_THREADS, tt = k / CC;
+            if (tt < m && mine) {
+                const float y = fmaf(my_d, us[k], ys[k]);
+                const float z = zrow ? zs[k] : in.at(t0 + c0 + tt, a.z_off + my_c);
+                out[(size_t)(t0 + c0 + tt) * a.inner + my_c] = from_f32<T>(y * silu_f(z));
             }
         }
     }
@@ -314,29 +338,76 @@ selective_scan_kernel(SelectiveArgs a, RowIn<float> in, StepArgs st, T* __restri
 
 // ------------------------------------------------------ read-out of the head scan
 // grid (tokens, norm groups): y = (num + D_h u) * silu(z) over its part's root mean square,
-// times the weight.
+// times the weight.  V consecutive channels (of one head) a thread at a time.
+template <int V>
+__device__ __forceinline__ void ld_v(const float* p, float (&o)[V]) {
+    if constexpr (V == 4) {
+        const float4 t = *reinterpret_cast<const float4*>(p);
+        o[0] = t.x, o[1] = t.y, o[2] = t.z, o[3] = t.w;
+    } else {
+        o[0] = *p;
+    }
+}
+__device__ __forceinline__ void st_v(float* p, const float (&a)[4]) {
+    *reinterpret_cast<float4*>(p) = make_float4(a[0], a[1], a[2], a[3]);
+}
+__device__ __forceinline__ void st_v(__nv_bfloat16* p, const float (&a)[4]) {
+    const __nv_bfloat162 lo = __floats2bfloat162_rn(a[0], a[1]), hi = __floats2bfloat162_rn(a[2], a[3]);
+    uint2 t;
+    t.x = *reinterpret_cast<const uint32_t*>(&lo);
+    t.y = *reinterpret_cast<const uint32_t*>(&hi);
+    *reinterpret_cast<uint2*>(p) = t;
+}
 template <typename T>
-__global__ void __launch_bounds__(256)
+__device__ __forceinline__ void st_v(T* p, const float (&a)[1]) { *p = from_f32<T>(a[0]); }
+
+template <typename T, int V>
+__global__ void __launch_bounds__(1024)
 ssd_out_kernel(const float* __restrict__ num, const float* __restrict__ u, long long ldu,
                const float* __restrict__ D, RowIn<float> in, int z_off, const float* __restrict__ weight,
                float eps, int inner, int dv, T* __restrict__ y) {
     pdl_wait();
     pdl_launch_next();
-    extern __shared__ float buf[];               // [inner / groups]
+    extern __shared__ __align__(16) float buf[]; // [inner / groups]
     __shared__ float red[33];
     const int t = blockIdx.x, width = inner / gridDim.y, c0 = blockIdx.y * width;
     float ss = 0.f;
-    for (int i = threadIdx.x; i < width; i += blockDim.x) {
+    for (int i = threadIdx.x * V; i < width; i += blockDim.x * V) {
         const int c = c0 + i;
-        const float v = fmaf(D[c / dv], u[(size_t)t * ldu + c], num[(size_t)t * inner + c]) *
-                        silu_f(in.at(t, z_off + c));
-        buf[i] = v;
-        ss = fmaf(v, v, ss);
+        float n[V], uu[V], z[V], v[V];
+        ld_v<V>(num + (size_t)t * inner + c, n);
+        ld_v<V>(u + (size_t)t * ldu + c, uu);
+        const float d = D[c / dv];
+        if (in.part) {
+            const float* p = in.part + (size_t)t * in.W + z_off + c;
+            ld_v<V>(p, z);
+#pragma unroll 4
+            for (int sp = 1; sp < in.n_splits; ++sp) {
+                float a[V];
+                ld_v<V>(p + (size_t)sp * in.split_stride, a);
+#pragma unroll
+                for (int k = 0; k < V; ++k) z[k] += a[k];
+            }
+        } else {
+            ld_v<V>(in.row + (size_t)t * in.ld + z_off + c, z);
+        }
+#pragma unroll
+        for (int k = 0; k < V; ++k) {
+            v[k] = fmaf(d, uu[k], n[k]) * silu_f(z[k]);
+            ss = fmaf(v[k], v[k], ss);
+        }
+        st_v(buf + i, v);
     }
     ss = block_sum(ss, red);
     const float r = 1.0f / sqrtf(ss / (float)width + eps);
-    for (int i = threadIdx.x; i < width; i += blockDim.x)
-        y[(size_t)t * inner + c0 + i] = from_f32<T>(buf[i] * r * weight[c0 + i]);
+    for (int i = threadIdx.x * V; i < width; i += blockDim.x * V) {
+        float v[V], w[V];
+        ld_v<V>(buf + i, v);                     // (a thread reads what it wrote)
+        ld_v<V>(weight + c0 + i, w);
+#pragma unroll
+        for (int k = 0; k < V; ++k) v[k] = v[k] * r * w[k];
+        st_v(y + (size_t)t * inner + c0 + i, v);
+    }
 }
 
 int row_of(RowIn<float>& in, const float* row, long long ld, const float* part, int n_splits, int T,
@@ -368,7 +439,7 @@ int launch_selective(const SelectiveArgs& a, const RowIn<float>& in, const StepA
                      T* out, cudaStream_t stream) {
     auto kern = selective_scan_kernel<T, NS, L>;
     constexpr int CC = SS_THREADS / L;
-    constexpr int smem = (2 * SS_CH * (2 * CC + 2 * NS * L) + 3 * SS_CH * CC) * (int)sizeof(float);
+    constexpr int smem = (2 * SS_CH * (3 * CC + 2 * NS * L) + 3 * SS_CH * CC) * (int)sizeof(float);
     static bool configured = false;
     if (smem > 48 * 1024 && !configured) {
         AGV_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
@@ -505,16 +576,23 @@ AGV_API int agv_ssd_out(const float* num, const float* u, long long ldu, const f
     RowIn<float> in;
     if (int rc = row_of(in, row, ld, part, n_splits, T, W)) return rc;
     const int width = inner / groups;
-    const int threads = width >= 1024 ? 256 : width >= 256 ? 128 : 64;
+    const bool vec = width % 4 == 0 && dv % 4 == 0 && z_off % 4 == 0 && ldu % 4 == 0 &&
+                     agv_aligned(num, 16) && agv_aligned(u, 16) && agv_aligned(weight, 16) &&
+                     agv_aligned(y, 16) &&
+                     (part ? W % 4 == 0 && agv_aligned(part, 16) : ld % 4 == 0 && agv_aligned(row, 16));
+    const int need = vec ? width / 4 : width;
+    // (few rows: all of a row's loads in one pass; many: several rows to an SM)
+    const int most = (long long)T * groups <= 296 ? 1024 : 256;
+    int threads = 32;
+    while (threads < most && threads < need) threads *= 2;
     const dim3 grid((unsigned)T, (unsigned)groups);
-    if (dtype == AGV_F32)
-        agv_launch(ssd_out_kernel<float>, grid, threads, smem, stream, num, u, ldu, D, in, z_off,
-                   weight, eps, inner, dv, (float*)y);
-    else if (dtype == AGV_BF16)
-        agv_launch(ssd_out_kernel<__nv_bfloat16>, grid, threads, smem, stream, num, u, ldu, D, in,
-                   z_off, weight, eps, inner, dv, (__nv_bfloat16*)y);
-    else
-        return agv_fail(-1, "ssd_out: unknown dtype %d", dtype);
+#define AGV_SO(TT, V)                                                                             \
+    agv_launch(ssd_out_kernel<TT, V>, grid, threads, smem, stream, num, u, ldu, D, in, z_off,     \
+               weight, eps, inner, dv, (TT*)y)
+    if (dtype == AGV_F32) { if (vec) AGV_SO(float, 4); else AGV_SO(float, 1); }
+    else if (dtype == AGV_BF16) { if (vec) AGV_SO(__nv_bfloat16, 4); else AGV_SO(__nv_bfloat16, 1); }
+    else return agv_fail(-1, "ssd_out: unknown dtype %d", dtype);
+#undef AGV_SO
     AGV_LAUNCH_OK("ssd_out_kernel");
     return 0;
 }

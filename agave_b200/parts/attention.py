@@ -104,8 +104,7 @@ class AttentionMixer:
         if self.keep_first and self.chunk is not None:
             raise ValueError("kept first keys go with a sliding window, not with a mask of blocks")
         if (self.conv_taps or self.out_gate) and (
-                spec.qk_norm is not None or self.q_temp is not None or self.value_mix is not None
-                or (self.position is not None and getattr(self.position, "interleaved", False))):
+                spec.qk_norm is not None or self.q_temp is not None or self.value_mix is not None):
             raise ValueError("a convolution on q, k and v or an output gate goes without q/k "
                              "norms, a query temperature or mixed values")
         if self.chunk is not None and (self.chunk < 1 or spec.window is not None):

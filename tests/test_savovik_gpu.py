@@ -534,7 +534,9 @@ MAMBA = [(72, scan(36, 5, 3, 2)), (128, scan(192, 16, 8, 4)), (96, scan(8, 1, 1,
          (40, scan(24, 128, 2, 4)), (40, scan(12, 200, 3, 2)), (64, scan(130, 3, 2, 4))]
 MAMBA2 = [(72, _m2(6, 10, 12, 3, 2, 3)), (128, _m2(4, 64, 64, 1, 1, 4)), (96, _m2(1, 16, 1, 1, 1, 1)),
           (76, _m2(5, 33, 18, 5, 1, 6)), (64, _m2(2, 7, 130, 2, 7, 2)), (48, _m2(8, 32, 48, 2, 4, 8)),
-          (64, _m2(2, 128, 256, 1, 2, 4)), (80, _m2(3, 8, 8, 3, 3, 2))]
+          (64, _m2(2, 128, 256, 1, 2, 4)), (80, _m2(3, 8, 8, 3, 3, 2)),
+          # (enough heads for the scan's form with two columns a lane, its last ones partly empty)
+          (32, _m2(100, 41, 20, 50, 4, 2))]
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
