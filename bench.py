@@ -41,7 +41,11 @@ Ramilorn decoder of equal width, heads, experts, layers and vocabulary.  ``--com
 sets the Kadavik decoder (attention with a convolution on q, k and v, a window behind which the
 first keys stay visible and an output gate, alternating with the matrix memory; routed experts
 with identity experts beside a gated shared one; a per-layer token input) beside the Bovozen
-decoder of equal width, heads, head size, experts, layers and vocabulary.
+decoder of equal width, heads, head size, experts, layers and vocabulary.  ``--compare savovik``
+sets the Savovik decoder (both branches of a layer from one norm with a gate each; chunked
+attention beside a selective scan, the head-wise state-space scan, windowed attention with
+capped scores) beside a Kadavik decoder of equal width, heads, head size, layers and vocabulary
+with dense feed-forwards of equal weight.
 """
 import argparse
 import json
@@ -372,7 +376,7 @@ def compare_configs_savovik(size):
             "rot": {"base": 1000000.0, "dims": d // 2,
                     "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}},
             "scale": d ** -0.5, "vdim": d}
-    par = {"left": left, "left_scale": 1.2, "right_scale": 0.8,
+    par = {"left": left, "left_scale": 1.1, "right_scale": 0.9,
            "right": {"conv": 4, "dt_rank": H // 16, "inner": 2 * H, "state": 16}}
     ssm = {"conv": 4, "groups": 1, "heads": 2 * H // 64, "norm_groups": 1, "state": N, "vdim": 64}
     kinds = [("parallel", par), ("mamba2", ssm), ("mamba2", ssm), ("attention", att)]

@@ -340,7 +340,7 @@ WINDOWED = [
     (210, 128, heads(8, 2, 64, 64, 0.13, size=100, rot=rotation(64, 1e4, 4.0), softcap=20.0)),
     (250, 96, heads(4, 2, 128, 64, 0.09, size=64, rot=rotation(64, 1e4, 8.0), softcap=2.0)),
     (70, 96, heads(2, 2, 24, 24, 0.3, size=1)),
-    (220, 80, heads(4, 4, 48, 48, 0.2, size=96, rot=rotation(48, 5e5), softcap=30.0)),
+    (220, 80, heads(4, 4, 48, 48, 0.2, size=90, rot=rotation(40, 2e5), softcap=18.0)),
     (140, 64, heads(2, 1, 32, 16, 0.25, softcap=1.0)),
 ]
 
@@ -533,7 +533,7 @@ MAMBA = [(72, scan(36, 5, 3, 2)), (128, scan(192, 16, 8, 4)), (96, scan(8, 1, 1,
          (76, scan(53, 24, 5, 7)), (64, scan(200, 33, 16, 3)), (48, scan(64, 8, 4, 8)),
          (40, scan(24, 128, 2, 4)), (40, scan(12, 200, 3, 2)), (64, scan(130, 3, 2, 4))]
 MAMBA2 = [(72, _m2(6, 10, 12, 3, 2, 3)), (128, _m2(4, 64, 64, 1, 1, 4)), (96, _m2(1, 16, 1, 1, 1, 1)),
-          (76, _m2(5, 33, 18, 5, 1, 6)), (64, _m2(2, 7, 130, 2, 7, 2)), (48, _m2(8, 32, 48, 2, 4, 8)),
+          (76, _m2(5, 33, 18, 5, 1, 6)), (64, _m2(2, 7, 130, 2, 7, 2)), (48, _m2(6, 40, 44, 2, 3, 8)),
           (64, _m2(2, 128, 256, 1, 2, 4)), (80, _m2(3, 8, 8, 3, 3, 2)),
           # (enough heads for the scan's form with two columns a lane, its last ones partly empty)
           (32, _m2(100, 41, 20, 50, 4, 2))]
