@@ -1,8 +1,8 @@
-from .base import (AttentionSpec, BlockSpec, ConfigError, DenseFeedForwardSpec, DistanceBiasSpec,
-                   GatedFeedForwardSpec, IdentityNormSpec, LatentAttentionSpec, LayerCall,
+from .base import (AttentionSpec, BlockSpec, ClampedGateSpec, ConfigError, DenseFeedForwardSpec,
+                   DistanceBiasSpec, GatedFeedForwardSpec, HeadDeltaSpec, IdentityNormSpec, LatentAttentionSpec, LayerCall,
                    LayerNormSpec, ModelSpec, NormSpec, ParallelBlockSpec, QueryTemperatureSpec,
                    RoutedFeedForwardSpec, RotarySpec, SelectiveScanSpec, SideBySideSpec,
-                   StateSpaceSpec, WavelengthScalingSpec, default_schedule)
+                   StateSpaceSpec, WavelengthScalingSpec, default_schedule, looped_schedule)
 from .registry import (load_config, read_config_json, register_architecture,
                        registered_architectures, resolve_architecture)
 from .gemma3 import Gemma3Config
@@ -11,6 +11,7 @@ from .zazerax import ZazeraxConfig
 from .bovozen import BovozenConfig
 from .kadavik import KadavikConfig
 from .savovik import SavovikConfig
+from .pubunex import PubunexConfig
 
 __all__ = [
     "AttentionSpec", "BlockSpec", "ConfigError", "GatedFeedForwardSpec", "LayerCall",
@@ -20,5 +21,6 @@ __all__ = [
     "resolve_architecture", "Gemma3Config", "ZazeraxConfig", "DenseFeedForwardSpec",
     "DistanceBiasSpec", "ParallelBlockSpec", "SelectiveScanSpec", "SideBySideSpec",
     "StateSpaceSpec", "IdentityNormSpec", "LatentAttentionSpec", "WavelengthScalingSpec",
-    "BovozenConfig", "KadavikConfig", "SavovikConfig",
+    "BovozenConfig", "KadavikConfig", "SavovikConfig", "PubunexConfig", "ClampedGateSpec",
+    "HeadDeltaSpec", "looped_schedule",
 ]

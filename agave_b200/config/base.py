@@ -182,6 +182,8 @@ class AttentionSpec:
     keep_all_keys: bool = False
     # biases added to the q, k and v projections (tensors ``q_proj.bias`` ...), before any norm
     qkv_bias: bool = False
+    # a bias added to the output projection (tensor ``o_proj.bias``)
+    out_bias: bool = False
     # scaled scores become softcap * tanh(score / softcap) before the mask; None: no cap
     softcap: Optional[float] = None
     # every value head is divided by its root mean square (this eps under the root, no weight)
@@ -201,7 +203,9 @@ class LatentAttentionSpec:
     (rot_dim wide) that all heads share.  Head a scores (q_a[:head_dim] . (W_uk c)_a +
     rot(q_a[head_dim:]) . kr) * scale and weighs (W_uv c)_a.  ``q_rank`` > 0: the queries
     come through a normed latent of that size too.  ``gate``: the heads' outputs are
-    multiplied by sigmoid(W_g x), "element" by element or one value per "head"."""
+    multiplied by sigmoid(W_g x), "element" by element or one value per "head".  ``sink``: a
+    learned logit per head (tensor ``sink``) whose exponential is one more term of the softmax
+    denominator (unscaled; nothing enters the weighted sum for it)."""
     kind: str = "latent_attention"
     n_heads: int = 0
     head_dim: int = 0            # unrotated part of a query / key head
@@ -213,6 +217,7 @@ class LatentAttentionSpec:
     eps: float = 1e-6
     position: Optional[RotarySpec] = None
     gate: Optional[str] = None
+    sink: bool = False
 
 
 @dataclass(frozen=True)
@@ -238,6 +243,29 @@ class ChannelDeltaSpec:
     gate_rank: int = 0
     eps: float = 1e-6
     unit_eps: float = 1e-6
+
+
+@dataclass(frozen=True)
+class HeadDeltaSpec:
+    """A recurrent mixer: the gated delta rule with one decay per head.
+
+    q, k (``n_qk_heads`` heads of ``head_dim``) and v (``n_heads`` heads of ``value_dim``)
+    pass a causal convolution over ``conv_taps`` tokens per channel and silu; q and k heads
+    become unit vectors (x / sqrt(sum x^2 + unit_eps)), q times head_dim ** -0.5.  Per head,
+    with beta = sigmoid(W_b x) and g = exp(-exp(A_log) * softplus(W_a x + dt_bias)):
+    S <- g S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q.  o / rms(o) (``eps``) * weight *
+    act(W_g x) feeds the output product, act = ``gate_activation`` ("silu" or "sigmoid").  The
+    state (S in 32-bit and the convolution's last conv_taps - 1 inputs) is a fixed size per
+    sequence."""
+    kind: str = "head_delta"
+    n_heads: int = 0
+    n_qk_heads: int = 0
+    head_dim: int = 0
+    value_dim: int = 0
+    conv_taps: int = 1
+    eps: float = 1e-6
+    unit_eps: float = 1e-6
+    gate_activation: str = "silu"
 
 
 @dataclass(frozen=True)
@@ -323,11 +351,20 @@ class TokenSideSpec:
 
 
 @dataclass(frozen=True)
+class ClampedGateSpec:
+    """The activation of a gated pair (g, u) with both held within bounds: g <- min(g, limit),
+    u <- clamp(u, -limit, limit), then g * sigmoid(alpha * g) * (u + 1)."""
+    limit: float
+    alpha: float = 1.702
+
+
+@dataclass(frozen=True)
 class GatedFeedForwardSpec:
     """down(act(gate x) * up x), dense (src/models/gemma3.zig:840-872)."""
     kind: str = "gated_dense"
     intermediate_size: int = 0
-    activation: str = "gelu_tanh"
+    # "gelu_tanh", "silu" or a ``ClampedGateSpec``
+    activation: object = "gelu_tanh"
 
 
 @dataclass(frozen=True)
@@ -350,7 +387,8 @@ class RoutedFeedForwardSpec:
     n_experts: int = 0
     top: int = 1
     intermediate_size: int = 0
-    activation: str = "silu"
+    # "gelu_tanh", "silu" or a ``ClampedGateSpec``
+    activation: object = "silu"
     n_groups: int = 1
     keep_groups: int = 1
     correction: bool = True
@@ -366,8 +404,14 @@ class RoutedFeedForwardSpec:
     # whose output is the feed-forward's input itself (times the weight)
     n_identity: int = 0
     # an expert of the same form that every token uses, of this width (0: none); its output is
-    # multiplied by sigmoid(w_sg . x), one number per token (tensor ``shared.gate.weight``)
+    # multiplied by sigmoid(w_sg . x), one number per token (tensor ``shared.gate.weight``),
+    # unless ``shared_gate`` is False; its activation is ``shared_activation`` (None: the
+    # experts')
     shared_size: int = 0
+    shared_gate: bool = True
+    shared_activation: Optional[object] = None
+    # a chosen expert's weight multiplies its input, expert(w x), instead of its output
+    weigh_input: bool = False
 
 
 @dataclass(frozen=True)
@@ -429,11 +473,14 @@ class LayerCall:
     whether this call appends to it (False: it reads what another call wrote).
     ``state``: the cache entry of the call's own fixed-size state where that is not
     ``cache`` (a call that reads another's keys and values and still has state of its own).
+    ``add_embedding``: the stream as it was before the first block is added to it right before
+    this call (a stack of blocks that runs again takes its input once more).
     """
     block: int
     cache: int
     writes_cache: bool = True
     state: Optional[int] = None
+    add_embedding: bool = False
 
 
 @dataclass(frozen=True)
@@ -469,3 +516,16 @@ class ModelSpec:
 
 def default_schedule(n_blocks: int) -> Tuple[LayerCall, ...]:
     return tuple(LayerCall(block=i, cache=i) for i in range(n_blocks))
+
+
+def looped_schedule(n_blocks: int, start: int, stop: int, times: int,
+                    add_embedding: bool = True) -> Tuple[LayerCall, ...]:
+    """Blocks start .. stop-1 run ``times`` times in a row, the others once; every call has a
+    cache entry of its own.  ``add_embedding``: each pass but the first begins with the stream
+    as it was before the first block added."""
+    order = [(i, False) for i in range(start)]
+    for t in range(times):
+        order += [(i, add_embedding and t > 0 and i == start) for i in range(start, stop)]
+    order += [(i, False) for i in range(stop, n_blocks)]
+    return tuple(LayerCall(block=i, cache=c, add_embedding=again)
+                 for c, (i, again) in enumerate(order))

@@ -11,11 +11,12 @@
 
 namespace {
 
-constexpr int JOIN_TERMS = 4;
+constexpr int JOIN_TERMS = 5;
 
 struct JoinTerm {
     const float* y32;          // [n_splits, R, H] or null
     const __nv_bfloat16* y16;  // [R, H] or null
+    long long row_stride;      // H, or 0: one row for all
     long long split_stride;
     int n_splits, gate;        // gate: index of its gate, or -1
     float mult;
@@ -116,9 +117,9 @@ gated_join_kernel(float* __restrict__ h, JoinArgs a, RowIn<float> gates,
         for (int j = 0; j < JOIN_TERMS; ++j) {
             if (j < a.n_terms) {
                 const JoinTerm& m = a.term[j];
-                const Pack<V> y = m.y32 ? sum_splits<V>(m.y32 + (size_t)t * H + i, m.n_splits,
+                const Pack<V> y = m.y32 ? sum_splits<V>(m.y32 + (size_t)t * m.row_stride + i, m.n_splits,
                                                         m.split_stride)
-                                        : ld_pack<V>(m.y16 + (size_t)t * H + i);
+                                        : ld_pack<V>(m.y16 + (size_t)t * m.row_stride + i);
 #pragma unroll
                 for (int k = 0; k < V; ++k) {
                     const float gk = m.gate < 0 ? 1.0f : m.gate == 0 ? g[0].v[k] : g[1].v[k];
@@ -149,8 +150,9 @@ gated_join_kernel(float* __restrict__ h, JoinArgs a, RowIn<float> gates,
 
 }  // namespace
 
-// Terms i < n_terms (at most 4): y[i] points to [n_splits[i], R, H] 32-bit sums (dtype[i] 0) or
-// [R, H] bfloat16 (dtype[i] 1), times mult[i], through gate gate[i] (-1: none).  gate_row / gate_part:
+// Terms i < n_terms (at most 5): y[i] points to [n_splits[i], R, H] 32-bit sums (dtype[i] 0) or
+// [R, H] bfloat16 (dtype[i] 1), or, with n_splits[i] 0, to one row [H] that every row takes (a
+// bias), times mult[i], through gate gate[i] (-1: none).  gate_row / gate_part:
 // the gates' logits [R, n_gates * H] 32-bit or partial sums of them; gate_bias [n_gates * H].  h [R,
 // H] or null; w_next [H] with x [R, H], or both null (or x alone: the sum as it is).
 AGV_API int agv_gated_join(float* h, int R, int H, int n_terms, const void* const* y,
@@ -172,15 +174,16 @@ AGV_API int agv_gated_join(float* h, int R, int H, int n_terms, const void* cons
                agv_aligned(gate_row, 16) && agv_aligned(gate_part, 16) && agv_aligned(gate_bias, 16) &&
                (!gate_row || gate_ld % 4 == 0);
     for (int i = 0; i < n_terms; ++i) {
-        AGV_REQUIRE(y[i] && n_splits[i] >= 1 && gate[i] >= -1 && gate[i] < n_gates,
+        AGV_REQUIRE(y[i] && n_splits[i] >= 0 && gate[i] >= -1 && gate[i] < n_gates,
                     "gated_join: term %d is incomplete", i);
-        AGV_REQUIRE(dtype[i] == AGV_F32 || (dtype[i] == AGV_BF16 && n_splits[i] == 1),
+        AGV_REQUIRE(dtype[i] == AGV_F32 || (dtype[i] == AGV_BF16 && n_splits[i] <= 1),
                     "gated_join: term %d must be 32-bit sums or one bfloat16 row", i);
         JoinTerm& m = a.term[i];
         m.y32 = dtype[i] == AGV_F32 ? (const float*)y[i] : nullptr;
         m.y16 = dtype[i] == AGV_BF16 ? (const __nv_bfloat16*)y[i] : nullptr;
         m.split_stride = (long long)R * H;
-        m.n_splits = n_splits[i], m.gate = gate[i], m.mult = mult[i];
+        m.row_stride = n_splits[i] ? H : 0;
+        m.n_splits = n_splits[i] ? n_splits[i] : 1, m.gate = gate[i], m.mult = mult[i];
         vec = vec && agv_aligned(y[i], 16);
     }
     const int W = n_gates * H;

@@ -11,18 +11,18 @@
 // (src/backend/kernels/cuda/gemv_bf16.zig:6-24, gemv_f32.zig:6-21); gated
 // activation src/backend/kernels/cuda/gelu_mul.zig:12-19 (here with tanhf).
 #include "common.cuh"
+#include "act.cuh"
 
 // (the squared relu, max(t, 0)^2, and the erf GELU, t/2 (1 + erf(t / sqrt 2)), go with the
 // plain product only)
-enum AgvActivation { AGV_ACT_GELU_TANH = 0, AGV_ACT_SILU = 1, AGV_ACT_RELU2 = 2, AGV_ACT_GELU_ERF = 3 };
-
 __device__ __forceinline__ float gelu_tanh_f(float t) {
     const float u = 0.7978845608028654f * (t + 0.044715f * t * t * t);
     return 0.5f * t * (1.0f + tanhf(u));
 }
 __device__ __forceinline__ float silu_f(float t) { return t / (1.0f + expf(-t)); }
-__device__ __forceinline__ float activate(float t, int act) {
-    return act == AGV_ACT_SILU ? silu_f(t) : gelu_tanh_f(t);
+__device__ __forceinline__ float activate(float g, float u, const GateAct& act) {
+    if (act.kind == AGV_ACT_CLAMPED) return clamped_gate(g, u, act);
+    return (act.kind == AGV_ACT_SILU ? silu_f(g) : gelu_tanh_f(g)) * u;
 }
 
 constexpr int BM = 64, BN = 64, BK = 16;
@@ -30,7 +30,7 @@ constexpr int BM = 64, BN = 64, BK = 16;
 template <typename TA, typename TW, typename TO, bool GATED>
 __global__ void __launch_bounds__(256)
 gemm_tn_kernel(const TA* __restrict__ A, const TW* __restrict__ W, const TW* __restrict__ W2,
-               TO* __restrict__ C, int M, int N, int K, long long lda, long long ldc, int act) {
+               TO* __restrict__ C, int M, int N, int K, long long lda, long long ldc, GateAct act) {
     pdl_wait();
     pdl_launch_next();
     __shared__ float As[BK][BM + 4];
@@ -83,9 +83,9 @@ gemm_tn_kernel(const TA* __restrict__ A, const TW* __restrict__ W, const TW* __r
             const int n = n0 + tx * 4 + j;
             if (n >= N) continue;
             float v = acc[i][j];
-            if (GATED) v = activate(v, act) * acc2[i][j];
-            else if (act == AGV_ACT_RELU2) { v = fmaxf(v, 0.f); v *= v; }
-            else if (act == AGV_ACT_GELU_ERF) v = 0.5f * v * (1.0f + erff(v * 0.7071067811865476f));
+            if (GATED) v = activate(v, acc2[i][j], act);
+            else if (act.kind == AGV_ACT_RELU2) { v = fmaxf(v, 0.f); v *= v; }
+            else if (act.kind == AGV_ACT_GELU_ERF) v = 0.5f * v * (1.0f + erff(v * 0.7071067811865476f));
             C[(size_t)m * ldc + n] = from_f32<TO>(v);
         }
     }
@@ -93,7 +93,7 @@ gemm_tn_kernel(const TA* __restrict__ A, const TW* __restrict__ W, const TW* __r
 
 template <typename TA, typename TW, typename TO>
 static int launch_gemm(const void* A, const void* W, const void* W2, void* C, int M, int N, int K,
-                       long long lda, long long ldc, int act, cudaStream_t stream) {
+                       long long lda, long long ldc, GateAct act, cudaStream_t stream) {
     dim3 grid((N + BN - 1) / BN, (M + BM - 1) / BM);
     if (W2)
         agv_launch(gemm_tn_kernel<TA, TW, TO, true>, grid, 256, 0, stream, (const TA*)A, (const TW*)W, (const TW*)W2, (TO*)C, M, N, K, lda, ldc, act);
@@ -108,10 +108,12 @@ static int launch_gemm(const void* A, const void* W, const void* W2, void* C, in
 // weights; out_dtype may be 32-bit for a bfloat16 product (logits).
 AGV_API int agv_linear_simt(const void* x, const void* w, const void* w2, void* out, int M, int N,
                             int K, long long lda, long long ldc, int in_dtype, int out_dtype,
-                            int act, cudaStream_t stream) {
+                            int act_kind, float act_alpha, float act_limit, cudaStream_t stream) {
+    const GateAct act{act_kind, act_alpha, act_limit};
     AGV_REQUIRE(M >= 0 && N > 0 && K > 0, "linear: bad sizes M=%d N=%d K=%d", M, N, K);
     AGV_REQUIRE(lda >= K && ldc >= N, "linear: row strides %lld, %lld shorter than rows", lda, ldc);
-    AGV_REQUIRE(act < AGV_ACT_RELU2 || !w2, "linear: the squared relu and the erf GELU go with a plain product");
+    AGV_REQUIRE(w2 ? gate_act_ok(act) : act_kind >= 0 && act_kind <= AGV_ACT_GELU_ERF,
+                "linear: activation %d does not go with this form of the product", act_kind);
     AGV_REQUIRE((long long)((M + BM - 1) / BM) <= 65535, "linear: M=%d exceeds the grid limit", M);
     if (M == 0) return 0;
     if (in_dtype == AGV_F32 && out_dtype == AGV_F32)

@@ -25,6 +25,7 @@
 // prompts (src/backend/cuda.zig:1569-1570).
 #include "common.cuh"
 #include "tcgen05.cuh"
+#include "act.cuh"
 #include "cache_write.cuh"
 #include <stdlib.h>
 #include <map>
@@ -70,6 +71,10 @@ __device__ __forceinline__ float gelu_tanh_fast(float t) {
     return 0.5f * t * (1.0f + th);
 }
 __device__ __forceinline__ float silu_fast(float t) { return __fdividef(t, 1.0f + __expf(-t)); }
+__device__ __forceinline__ float gated_fast(float g, float u, const GateAct& act) {
+    if (act.kind == AGV_ACT_CLAMPED) return clamped_gate_fast(g, u, act);
+    return (act.kind == AGV_ACT_SILU ? silu_fast(g) : gelu_tanh_fast(g)) * u;
+}
 // The activation a plain product may carry: 2 the squared relu, 3 the erf GELU.
 __device__ __forceinline__ float plain_act(float t, int act) {
     if (act == 2) { t = fmaxf(t, 0.f); return t * t; }
@@ -129,7 +134,7 @@ __global__ void __launch_bounds__(GEMM_THREADS, 1)
 gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_w,
                     const __grid_constant__ CUtensorMap map_w2,
                     const __grid_constant__ CUtensorMap map_x, TO* __restrict__ out, int T, int N,
-                    int K, long long ldc, long long split_stride, int kb_per_split, int act,
+                    int K, long long ldc, long long split_stride, int kb_per_split, GateAct act,
                     int cluster_reduce, int* __restrict__ argmax_out) {
     pdl_launch_next();
     using TL = Tile<BN, MODE, SLIM>;
@@ -340,8 +345,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_w,
                             if (n < T) {
                                 const float gv = __uint_as_float(r[j]);
                                 const float uv = xchg[(c + j) * 64 + quarter * 32 + lane];
-                                store_out<TO>(obase + (size_t)n * ldc + f,
-                                              (act == 1 ? silu_fast(gv) : gelu_tanh_fast(gv)) * uv);
+                                store_out<TO>(obase + (size_t)n * ldc + f, gated_fast(gv, uv, act));
                             }
                         }
                     }
@@ -365,8 +369,8 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_w,
                     for (int j = 0; j < 16; ++j) {
                         float v = __uint_as_float(r[j]);
                         if (GATED)
-                            v = (act == 1 ? silu_fast(v) : gelu_tanh_fast(v)) * __uint_as_float(u[j]);
-                        else if (MODE == 0 && act >= 2) v = plain_act(v, act);
+                            v = gated_fast(v, __uint_as_float(u[j]), act);
+                        else if (MODE == 0 && act.kind >= 2) v = plain_act(v, act.kind);
                         store_out<TO>(ctile + (c + j) * TILE_M + fl, v);
                     }
                 }
@@ -449,8 +453,8 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_w,
                         acc += inbox[((size_t)q * BN + n) * rows + jl];
                         if (HALF) up += inbox[((size_t)q * BN + n) * rows + per + jl];
                     }
-                    if (HALF) acc = (act == 1 ? silu_fast(acc) : gelu_tanh_fast(acc)) * up;
-                    else if (MODE == 0 && act >= 2) acc = plain_act(acc, act);
+                    if (HALF) acc = gated_fast(acc, up, act);
+                    else if (MODE == 0 && act.kind >= 2) acc = plain_act(acc, act.kind);
                     store_out<TO>(gout + (size_t)(n0 + n) * ldc + m0 + fl, acc);
                 }
             }
@@ -476,9 +480,9 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_w,
                         float up = 0.f;
 #pragma unroll
                         for (int q = 0; q < 8; ++q) up += pu[q];
-                        acc = (act == 1 ? silu_fast(acc) : gelu_tanh_fast(acc)) * up;
-                    } else if (MODE == 0 && act >= 2) {
-                        acc = plain_act(acc, act);
+                        acc = gated_fast(acc, up, act);
+                    } else if (MODE == 0 && act.kind >= 2) {
+                        acc = plain_act(acc, act.kind);
                     }
                     store_out<TO>(gout + (size_t)(n0 + n) * ldc + m0 + fl, acc);
                 }
@@ -711,7 +715,7 @@ gemm_tcgen05_persistent_kernel(const __grid_constant__ CUtensorMap map_w,
                                const __grid_constant__ CUtensorMap map_w2,
                                const __grid_constant__ CUtensorMap map_x, TO* __restrict__ out,
                                int T, int N, int K, long long ldc, long long split_stride,
-                               int splits, int kb_per_split, int act,
+                               int splits, int kb_per_split, GateAct act,
                                const __grid_constant__ QkvEpilogue qe) {
     pdl_launch_next();
     using TL = PTile<BN, MODE>;
@@ -893,7 +897,12 @@ gemm_tcgen05_persistent_kernel(const __grid_constant__ CUtensorMap map_w,
             auto work = [&](const uint32_t (&r)[16], const uint32_t (&u)[16], int c) {
                 if constexpr (GATED) {
                     float v[16];
-                    if (act == 1) {
+                    if (act.kind == AGV_ACT_CLAMPED) {
+#pragma unroll
+                        for (int j = 0; j < 16; ++j)
+                            v[j] = clamped_gate_fast(__uint_as_float(r[j]), __uint_as_float(u[j]),
+                                                     act);
+                    } else if (act.kind == AGV_ACT_SILU) {
 #pragma unroll
                         for (int j = 0; j < 16; ++j)
                             v[j] = silu_fast(__uint_as_float(r[j])) * __uint_as_float(u[j]);
@@ -921,23 +930,15 @@ gemm_tcgen05_persistent_kernel(const __grid_constant__ CUtensorMap map_w,
                     return;
                 }
                 if (GATED) {
-                    if (act == 1) {
 #pragma unroll
-                        for (int j = 0; j < 16; ++j)
-                            store_out<TO>(wst + j * 32 + lane, silu_fast(__uint_as_float(r[j])) *
-                                                                   __uint_as_float(u[j]));
-                    } else {
-#pragma unroll
-                        for (int j = 0; j < 16; ++j)
-                            store_out<TO>(wst + j * 32 + lane,
-                                          gelu_tanh_fast(__uint_as_float(r[j])) *
-                                              __uint_as_float(u[j]));
-                    }
-                } else if (MODE == 0 && act >= 2) {
+                    for (int j = 0; j < 16; ++j)
+                        store_out<TO>(wst + j * 32 + lane,
+                                      gated_fast(__uint_as_float(r[j]), __uint_as_float(u[j]), act));
+                } else if (MODE == 0 && act.kind >= 2) {
                     // plain product with an activation on it
 #pragma unroll
                     for (int j = 0; j < 16; ++j)
-                        store_out<TO>(wst + j * 32 + lane, plain_act(__uint_as_float(r[j]), act));
+                        store_out<TO>(wst + j * 32 + lane, plain_act(__uint_as_float(r[j]), act.kind));
                 } else {
 #pragma unroll
                     for (int j = 0; j < 16; ++j)
@@ -1072,7 +1073,7 @@ gemm_tcgen05_pair_gated_kernel(const __grid_constant__ CUtensorMap map_w,
                                const __grid_constant__ CUtensorMap map_w2,
                                const __grid_constant__ CUtensorMap map_x,
                                __nv_bfloat16* __restrict__ out, int T, int N, int K, long long ldc,
-                               int act) {
+                               GateAct act) {
     pdl_launch_next();
     typedef __nv_bfloat16 TO;
     extern __shared__ uint8_t smem_raw[];
@@ -1224,7 +1225,11 @@ gemm_tcgen05_pair_gated_kernel(const __grid_constant__ CUtensorMap map_w,
             };
             auto work = [&](const uint32_t (&r)[16], const uint32_t (&u)[16], int c) {
                 float v[16];
-                if (act == 1) {
+                if (act.kind == AGV_ACT_CLAMPED) {
+#pragma unroll
+                    for (int j = 0; j < 16; ++j)
+                        v[j] = clamped_gate_fast(__uint_as_float(r[j]), __uint_as_float(u[j]), act);
+                } else if (act.kind == AGV_ACT_SILU) {
 #pragma unroll
                     for (int j = 0; j < 16; ++j)
                         v[j] = silu_fast(__uint_as_float(r[j])) * __uint_as_float(u[j]);
@@ -1322,7 +1327,7 @@ int make_map(CUtensorMap* out, const void* ptr, long long rows, long long K, lon
 template <int BN, int MODE, typename TO, int SLIM = 0>
 int launch(const CUtensorMap& mw, const CUtensorMap& mw2, const CUtensorMap& mx, void* out, int T,
            int N, int K, long long ldc, long long split_stride, int splits, int kb_per_split,
-           int act, int cluster_reduce, cudaStream_t stream, int* argmax_out = nullptr) {
+           GateAct act, int cluster_reduce, cudaStream_t stream, int* argmax_out = nullptr) {
     using TL = Tile<BN, MODE, SLIM>;
     static_assert(MODE != 0 || BN * RED_LD * 4 <= TL::STAGES * TL::STAGE_BYTES,
                   "a partial tile must fit the ring of stages");
@@ -1353,7 +1358,7 @@ int launch(const CUtensorMap& mw, const CUtensorMap& mw2, const CUtensorMap& mx,
 template <int BN, int MODE, typename TO>
 int launch_persistent(const CUtensorMap& mw, const CUtensorMap& mw2, const CUtensorMap& mx,
                       void* out, int T, int N, int K, long long ldc, long long split_stride,
-                      int splits, int kb_per_split, int act, cudaStream_t stream,
+                      int splits, int kb_per_split, GateAct act, cudaStream_t stream,
                       const QkvEpilogue& qe = QkvEpilogue{}) {
     using TL = PTile<BN, MODE>;
     auto kern = gemm_tcgen05_persistent_kernel<BN, MODE, TO>;
@@ -1378,7 +1383,7 @@ int launch_persistent(const CUtensorMap& mw, const CUtensorMap& mw2, const CUten
 }
 
 int launch_pair_gated(const CUtensorMap& mw, const CUtensorMap& mw2, const CUtensorMap& mx,
-                      void* out, int T, int N, int K, long long ldc, int act, cudaStream_t stream) {
+                      void* out, int T, int N, int K, long long ldc, GateAct act, cudaStream_t stream) {
     auto kern = gemm_tcgen05_pair_gated_kernel;
     static bool configured = false;
     static int sms = 0;
@@ -1403,7 +1408,7 @@ int launch_pair_gated(const CUtensorMap& mw, const CUtensorMap& mw2, const CUten
 template <int MODE, typename TO>
 int launch_bn(int bn, const CUtensorMap& mw, const CUtensorMap& mw2, const CUtensorMap& mx,
               void* out, int T, int N, int K, long long ldc, long long split_stride, int splits,
-              int kb_per_split, int act, int cluster_reduce, cudaStream_t stream) {
+              int kb_per_split, GateAct act, int cluster_reduce, cudaStream_t stream) {
 #define AGV_BN_CASE(B)                                                                          \
     case B:                                                                                      \
         return launch<B, MODE, TO>(mw, mw2, mx, out, T, N, K, ldc, split_stride, splits,         \
@@ -1440,8 +1445,10 @@ AGV_API int agv_linear_tc_supported(int N, int K, long long lda) {
 // memory in rank order, and out is [splits / c, T, N] (a plain [T, N] when
 // splits == c; bf16 allowed then).  token_tile 0 lets the launcher choose.
 AGV_API int agv_linear_tc(const void* x, const void* w, const void* w2, void* out, int T, int N,
-                          int K, long long lda, long long ldc, int out_dtype, int act, int splits,
-                          int cluster, int token_tile, cudaStream_t stream) {
+                          int K, long long lda, long long ldc, int out_dtype, int act_kind,
+                          float act_alpha, float act_limit, int splits, int cluster,
+                          int token_tile, cudaStream_t stream) {
+    const GateAct act{act_kind, act_alpha, act_limit};
     AGV_REQUIRE(T >= 0 && N > 0 && K > 0, "linear: bad sizes T=%d N=%d K=%d", T, N, K);
     AGV_REQUIRE(K % 8 == 0 && lda % 8 == 0, "linear: the tensor-core kernel needs K (%d) and the "
                 "row stride (%lld) to be multiples of 8", K, lda);
@@ -1451,7 +1458,9 @@ AGV_API int agv_linear_tc(const void* x, const void* w, const void* w2, void* ou
     AGV_REQUIRE(splits >= 1, "linear: splits must be >= 1");
     // act 2 (the squared relu) and 3 (the erf GELU) belong to the plain product and need a
     // finished sum
-    AGV_REQUIRE(act < 2 || (!w2 && (splits == 1 || splits == cluster)),
+    AGV_REQUIRE(w2 ? gate_act_ok(act) : act_kind >= 0 && act_kind <= AGV_ACT_GELU_ERF,
+                "linear: activation %d does not go with this form of the product", act_kind);
+    AGV_REQUIRE(w2 || act_kind < 2 || splits == 1 || splits == cluster,
                 "linear: the squared relu and the erf GELU go with a plain product whose sum is "
                 "finished in the kernel (one range of K, or one cluster's)");
     AGV_REQUIRE(splits == 1 || !w2 || (cluster == splits && T <= 64),
@@ -1586,8 +1595,8 @@ AGV_API int agv_linear_tc_argmax(const void* x, const void* w, int* out_idx, int
     if (int rc = make_map(&mx, x, T, K, lda, bn)) return rc;
 #define AGV_ARGMAX_CASE(B)                                                                      \
     case B:                                                                                      \
-        rc = launch<B, 0, float>(mw, mw, mx, nullptr, T, N, K, N, 0, 1, kb_total, 0, 0, stream,  \
-                                 out_idx);                                                       \
+        rc = launch<B, 0, float>(mw, mw, mx, nullptr, T, N, K, N, 0, 1, kb_total, GateAct{}, 0, \
+                                 stream, out_idx);                                                       \
         break
     int rc = -1;
     switch (bn) {
@@ -1647,7 +1656,7 @@ AGV_API int agv_qkv_prefill_tc(const void* x, const void* w, int T, int K, long 
                    VtWrite{(__nv_bfloat16*)vt, vt_ld, cu_seqlens, seq_index}};
     const int kb_total = (K + TILE_K - 1) / TILE_K;
     return launch_persistent<128, 3, __nv_bfloat16>(mw, mw, mx, nullptr, T, N, K, 0, 0, 1, kb_total,
-                                                    0, stream, qe);
+                                                    GateAct{}, stream, qe);
 }
 
 // The number of partial sums agv_linear_tc will really write for these sizes.

@@ -33,9 +33,9 @@ int agv_rope_table(const int*, float*, float*, int, int, double, double, cudaStr
 int agv_norm_residual(float*, const void*, int, int, long long, const float*, const float*, void*,
                       int, const int*, int, int, float, float, int, cudaStream_t);
 int agv_linear_simt(const void*, const void*, const void*, void*, int, int, int, long long,
-                    long long, int, int, int, cudaStream_t);
+                    long long, int, int, int, float, float, cudaStream_t);
 int agv_linear_tc(const void*, const void*, const void*, void*, int, int, int, long long, long long,
-                  int, int, int, int, int, cudaStream_t);
+                  int, int, float, float, int, int, int, cudaStream_t);
 int agv_linear_tc_splits(int, int);
 int agv_gemv_few_supported(int, int, int, long long, int);
 int agv_gemv_few(const void*, const void*, int, int, int, const void*, long long, const float*, float*,
@@ -226,13 +226,14 @@ struct Run {
             plan_splits(T, N, K, cheap, &groups, &c);
             void* out = ar.take((size_t)groups * T * N * 4);
             if (!dry())
-                did(agv_linear_tc(x, w, nullptr, out, T, N, K, lda, N, AGV_F32, 0,
+                did(agv_linear_tc(x, w, nullptr, out, T, N, K, lda, N, AGV_F32, 0, 0.f, 0.f,
                                   groups * (c > 1 ? c : 1), c, 0, stream));
             return {out, groups};
         }
         void* out = ar.take((size_t)T * N * esz());
         if (!dry())
-            did(agv_linear_simt(x, w, nullptr, out, T, N, K, lda, N, m.dtype, m.dtype, 0, stream));
+            did(agv_linear_simt(x, w, nullptr, out, T, N, K, lda, N, m.dtype, m.dtype, 0, 0.f, 0.f,
+                                stream));
         return {out, 0};
     }
 
@@ -390,11 +391,11 @@ struct Run {
                     const int tiles = (b.ff + 63) / 64, kb = (H + 63) / 64;
                     c = (tiles * 4 <= sms && kb >= 8) ? 4 : (tiles * 2 <= 2 * sms && kb >= 4) ? 2 : 0;
                 }
-                did(agv_linear_tc(x, b.w_gate, b.w_up, z, T, b.ff, H, H, b.ff, AGV_BF16, b.act,
+                did(agv_linear_tc(x, b.w_gate, b.w_up, z, T, b.ff, H, H, b.ff, AGV_BF16, b.act, 0.f, 0.f,
                                   c > 1 ? c : 1, c, 0, stream));
             } else {
                 did(agv_linear_simt(x, b.w_gate, b.w_up, z, T, b.ff, H, H, b.ff, m.dtype, m.dtype,
-                                    b.act, stream));
+                                    b.act, 0.f, 0.f, stream));
             }
         }
         return linear_partial(z, b.ff, b.w_down, H, b.ff, T, false);
@@ -536,10 +537,10 @@ struct Run {
                     ++launches;               // the product and the kernel that reads its keys out
                 } else if (tc_ok(xn, H, m.head_w, H)) {
                     did(agv_linear_tc(xn, m.head_w, nullptr, s.logits, s.n_rows, m.V, H, H, m.V,
-                                      AGV_F32, 0, 1, 0, 0, stream));
+                                      AGV_F32, 0, 0.f, 0.f, 1, 0, 0, stream));
                 } else {
                     did(agv_linear_simt(xn, m.head_w, nullptr, s.logits, s.n_rows, m.V, H, H, m.V,
-                                        m.dtype, AGV_F32, 0, stream));
+                                        m.dtype, AGV_F32, 0, 0.f, 0.f, stream));
                 }
             }
         }

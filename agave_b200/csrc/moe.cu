@@ -19,18 +19,19 @@
 // Grouped products: out[pos, :] = a[src(pos), :] * W[e(tile)]^T, plain, or the gated pair
 // act(a Wg^T) * (a Wu^T); a row of the result can be scaled and scattered (the down
 // product leaves w_pair * y at [choice, token, :], which the join that follows adds over
-// the choices in order).  Each output element is one dot product accumulated in ascending
+// the choices in order).  On the gated pair the scale multiplies the row's two sums before the
+// activation: what the experts make of w_pair * x, without x being scaled and rounded.  Each output element is one dot product accumulated in ascending
 // k in 32-bit: a token's result does not depend on its company.
 #include "common.cuh"
+#include "act.cuh"
 
 namespace {
 
-enum { MOE_ACT_GELU_TANH = 0, MOE_ACT_SILU = 1 };
-
-__device__ __forceinline__ float moe_act(float t, int act) {
-    if (act == MOE_ACT_SILU) return t / (1.0f + expf(-t));
-    const float u = 0.7978845608028654f * (t + 0.044715f * t * t * t);
-    return 0.5f * t * (1.0f + tanhf(u));
+__device__ __forceinline__ float moe_act(float g, float u, const GateAct& act) {
+    if (act.kind == AGV_ACT_CLAMPED) return clamped_gate(g, u, act);
+    if (act.kind == AGV_ACT_SILU) return g / (1.0f + expf(-g)) * u;
+    const float v = 0.7978845608028654f * (g + 0.044715f * g * g * g);
+    return 0.5f * g * (1.0f + tanhf(v)) * u;
 }
 
 constexpr int RT_WARPS = 4;
@@ -389,7 +390,7 @@ moe_grouped_kernel(const TA* __restrict__ A, long long lda, const int* __restric
                    const int* __restrict__ tok, const TW* __restrict__ W,
                    const TW* __restrict__ W2, TO* __restrict__ C, long long ldc,
                    const int* __restrict__ c_index, const float* __restrict__ c_scale,
-                   const int* __restrict__ tile_e, int N, int K, int act, int sub) {
+                   const int* __restrict__ tile_e, int N, int K, GateAct act, int sub) {
     pdl_wait();
     pdl_launch_next();
     const int e = tile_e[blockIdx.y / sub];
@@ -456,9 +457,9 @@ moe_grouped_kernel(const TA* __restrict__ A, long long lda, const int* __restric
         for (int j = 0; j < 4; ++j) {
             const int n = n0 + tx * 4 + j;
             if (n >= N) continue;
-            float v = acc[i][j];
-            if (GATED) v = moe_act(v, act) * acc2[i][j];
-            C[crow * ldc + n] = from_f32<TO>(v * sc);
+            float v = acc[i][j] * sc;
+            if (GATED) v = moe_act(v, acc2[i][j] * sc, act);
+            C[crow * ldc + n] = from_f32<TO>(v);
         }
     }
 }
@@ -604,14 +605,18 @@ AGV_API int agv_moe_plan(const int* ids, const float* wts, int T, int top, int E
 
 // The grouped product over a plan.  a: rows of stride lda (a_index null: row = sorted
 // position); tile: the plan's rows per tile; w (and w2 for the gated form): [E, N, K] dense; c: rows of stride ldc at
-// c_index[pos] (null: pos), times c_scale[pos] (null: 1).  in_dtype: a and the weights;
-// out_dtype: c.
+// c_index[pos] (null: pos), times c_scale[pos] (null: 1; the gated form scales the two sums
+// before the activation).  in_dtype: a and the weights; out_dtype: c.  act, act_alpha and
+// act_limit: the gated form's activation (act.cuh).
 AGV_API int agv_moe_grouped(const void* a, long long lda, const int* a_index, const int* tok,
                             const void* w, const void* w2, void* c, long long ldc,
                             const int* c_index, const float* c_scale, const int* tile_e,
                             int n_tiles, int tile, int N, int K, int in_dtype, int out_dtype,
-                            int act, cudaStream_t stream) {
+                            int act_kind, float act_alpha, float act_limit,
+                            cudaStream_t stream) {
+    const GateAct act{act_kind, act_alpha, act_limit};
     AGV_REQUIRE(n_tiles >= 0 && N > 0 && K > 0, "moe_grouped: bad sizes");
+    AGV_REQUIRE(!w2 || gate_act_ok(act), "moe_grouped: unknown activation %d", act_kind);
     AGV_REQUIRE(tile >= GM && tile % GM == 0, "moe_grouped: tiles of %d rows (a multiple of %d)",
                 tile, GM);
     const int sub = tile / GM;

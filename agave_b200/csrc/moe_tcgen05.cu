@@ -9,7 +9,8 @@
 // swizzle into a ring of stages, the products accumulate in tensor memory, and four
 // warps read the accumulator back, one output feature per thread, and pass the tile
 // through shared memory so that rows leave in 16-byte pieces:
-//   gated:  z[pos, f] = act(gate) * up, two accumulators side by side, bfloat16 out;
+//   gated:  z[pos, f] = act(gate, up), two accumulators side by side (times the pair's weight
+//           before the activation, where it multiplies an expert's input), bfloat16 out;
 //   plain:  out[dst[pos], f] = w[pos] * acc, 32-bit out (the down product, scattered to
 //           [choice, token] and scaled by the pair's weight).
 // Rows of padding (tok[pos] < 0) are computed and dropped.  The left operand's rows must
@@ -20,6 +21,7 @@
 // requested before the wait for the kernels before; every wait on a barrier is bounded
 // and leaves a code for agv_moe_tc_status.
 #include "tcgen05.cuh"
+#include "act.cuh"
 #include <type_traits>
 
 namespace {
@@ -44,12 +46,13 @@ struct MTile {
     static constexpr int SMEM = STAGES * STAGE_BYTES + 1024 /*align*/ + 2048 /*barriers, rows*/;
 };
 
-__device__ __forceinline__ float mt_act(float t, int act) {
-    if (act == 1) return __fdividef(t, 1.0f + __expf(-t));
-    const float u = 0.7978845608028654f * (t + 0.044715f * t * t * t);
+__device__ __forceinline__ float mt_act(float g, float u, const GateAct& act) {
+    if (act.kind == AGV_ACT_CLAMPED) return clamped_gate_fast(g, u, act);
+    if (act.kind == AGV_ACT_SILU) return __fdividef(g, 1.0f + __expf(-g)) * u;
+    const float v = 0.7978845608028654f * (g + 0.044715f * g * g * g);
     float th;
-    asm("tanh.approx.f32 %0, %1;" : "=f"(th) : "f"(u));
-    return 0.5f * t * (1.0f + th);
+    asm("tanh.approx.f32 %0, %1;" : "=f"(th) : "f"(v));
+    return 0.5f * g * (1.0f + th) * u;
 }
 
 template <bool GATED, int MT_N>
@@ -59,7 +62,7 @@ moe_grouped_tc_kernel(const __grid_constant__ CUtensorMap map_w,
                       const __grid_constant__ CUtensorMap map_a, void* __restrict__ out,
                       long long ldc, const int* __restrict__ tok, const int* __restrict__ c_index,
                       const float* __restrict__ c_scale, const int* __restrict__ tile_e, int N,
-                      int K, int act) {
+                      int K, GateAct act) {
     pdl_launch_next();
     pdl_wait();                                    // the plan is the work of kernels before
     const int e = tile_e[blockIdx.y];
@@ -194,7 +197,9 @@ moe_grouped_tc_kernel(const __grid_constant__ CUtensorMap map_w,
                 for (int j = 0; j < 16; ++j) {
                     float v = __uint_as_float(r[j]);
                     if constexpr (GATED) {
-                        v = mt_act(v, act) * __uint_as_float(u[j]);
+                        float w = __uint_as_float(u[j]);
+                        if (c_scale) v *= s_scale[c + j], w *= s_scale[c + j];
+                        v = mt_act(v, w, act);
                         ctile[(c + j) * MT_M + fl] = __float2bfloat16_rn(v);
                     } else {
                         ctile[(c + j) * MT_M + fl] = v * s_scale[c + j];
@@ -297,13 +302,16 @@ AGV_API int agv_moe_gather_rows(const void* x, long long ldx, const int* tok, vo
 
 // a: [rows, K] bfloat16 in sorted order (row stride lda); w (and w2 for the gated form):
 // [E, N, K] bfloat16 dense; tok, tile_e: the plan.  Gated: c [rows, N] bfloat16 rows of stride
-// ldc at the sorted positions.  Plain: c 32-bit, row c_index[pos] (null: pos) times
+// ldc at the sorted positions, c_scale[pos] (if not null) times the two sums before the
+// activation.  Plain: c 32-bit, row c_index[pos] (null: pos) times
 // c_scale[pos] (null: 1).  tile: the plan's rows per tile, 64 or 128.
 AGV_API int agv_moe_grouped_tc(const void* a, long long lda, int rows, const int* tok,
                                const void* w, const void* w2, int E, void* c, long long ldc,
                                const int* c_index, const float* c_scale, const int* tile_e,
-                               int n_tiles, int tile, int N, int K, int act,
-                               cudaStream_t stream) {
+                               int n_tiles, int tile, int N, int K, int act_kind,
+                               float act_alpha, float act_limit, cudaStream_t stream) {
+    const GateAct act{act_kind, act_alpha, act_limit};
+    AGV_REQUIRE(!w2 || gate_act_ok(act), "moe_grouped_tc: unknown activation %d", act_kind);
     AGV_REQUIRE(tile == 64 || tile == 128, "moe_grouped_tc: tiles of %d rows (64 or 128)", tile);
     AGV_REQUIRE(n_tiles >= 0 && E > 0 && rows >= n_tiles * tile, "moe_grouped_tc: bad sizes");
     AGV_REQUIRE(agv_moe_grouped_tc_supported(N, K, lda), "moe_grouped_tc: K (%d) and the row "

@@ -3,7 +3,7 @@
 //  * agv_ssm_conv: from a token's row of the stacked input projection (32-bit, or 32-bit partial
 //    sums over ranges of K), channels off .. off + C: a causal convolution over time, channel by
 //    channel (``taps`` weights a channel, the last one the current token's; zeros before the
-//    start of a sequence), a bias and silu.  The convolution's inputs of earlier steps are part
+//    start of a sequence), a bias (or none) and silu.  The convolution's inputs of earlier steps are part
 //    of the sequence's fixed-size state: a ring by position (position p in row p % (taps - 1)).
 //    Beside them, columns dt_off .. + n_dt may hold one step size per head: dt = softplus(dt +
 //    bias), which leaves as the pair (exp(neg_a dt), dt) a scan with one decay per head wants.
@@ -87,7 +87,7 @@ ssm_conv_kernel(RowIn<float> in, int n_tokens, int off, int C, StepArgs st,
     float wv[TAPS], xs[R + RING];
 #pragma unroll
     for (int j = 0; j < TAPS; ++j) wv[j] = w[(size_t)c * TAPS + j];
-    const float b = bias[c];
+    const float b = bias ? bias[c] : 0.f;
     long long ld;
     if (const float* src = in.single(ld)) {                    // (all loads in flight at once)
 #pragma unroll
@@ -454,7 +454,7 @@ int launch_selective(const SelectiveArgs& a, const RowIn<float>& in, const StepA
 }  // namespace
 
 // row / part: the stacked projection [T, W] 32-bit (row stride ld) or [n_splits, T, W] partial
-// sums.  conv_w [C, taps], conv_b [C] 32-bit.  out [T, C] 32-bit and, if not null, rounded [T, C]
+// sums.  conv_w [C, taps], conv_b [C] (or null) 32-bit.  out [T, C] 32-bit and, if not null, rounded [T, C]
 // in dtype.  state: the ring, (taps - 1) * C values per slot from state_off on.  n_dt > 0: coef
 // [T, n_dt, 2] receives (exp(neg_a dt), dt) of the columns dt_off ..
 AGV_API int agv_ssm_conv(const float* row, long long ld, const float* part, int n_splits, int T,

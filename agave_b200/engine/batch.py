@@ -52,6 +52,9 @@ class StepContext:
     # the tokens' rows of the table of per-layer token inputs, 32-bit [T, width], gathered
     # once a step for all layers (None: the model has no such table)
     token_side_rows: Optional[torch.Tensor] = None
+    # what the running block adds to the stream besides its branches, 32-bit [T, hidden] (None:
+    # nothing; the decoder sets it where the run order asks for the embedding once more)
+    join_extra: Optional[torch.Tensor] = None
 
     def new(self, *shape, dtype=None) -> torch.Tensor:
         return torch.empty(shape, dtype=dtype or self.dtype, device=self.device)

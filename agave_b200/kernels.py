@@ -18,7 +18,21 @@ from . import perf as _perf_mod
 from .csrc import build as _build
 
 F32, BF16 = 0, 1
-ACT = {"gelu_tanh": 0, "silu": 1, "relu2": 2, "gelu_erf": 3}   # 2, 3: on a plain product only
+ACT = {"gelu_tanh": 0, "silu": 1, "relu2": 2, "gelu_erf": 3,   # 2, 3: on a plain product only
+       "clamped": 4}                                          # 4: on a gated pair only
+
+
+def _act(activation, w2):
+    """(kind, alpha, limit) of an activation as the products take it: a name, or for a gated
+    pair ("clamped", alpha, limit): with g <- min(g, limit) and u <- clamp(u, -limit, limit),
+    g * sigmoid(alpha * g) * (u + 1)."""
+    if isinstance(activation, str):
+        kind, alpha, limit = activation, 0.0, 0.0
+    else:
+        kind, alpha, limit = activation
+    if (kind == "clamped") and (w2 is None or not limit > 0):
+        raise KernelError("the clamped activation goes with a gated pair and a positive limit")
+    return ACT[kind], ctypes.c_float(alpha), ctypes.c_float(limit)
 
 _lib = None
 _lock = threading.Lock()
@@ -367,12 +381,15 @@ def moe_plan(ids: torch.Tensor, wts: torch.Tensor, n_experts: int, tile: int = 0
 
 
 def moe_grouped(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, plan: MoePlan,
-                w2: Optional[torch.Tensor] = None, activation: str = "silu",
-                gather: bool = False, scatter: bool = False, op: str = "experts") -> None:
+                w2: Optional[torch.Tensor] = None, activation="silu",
+                gather: bool = False, scatter: bool = False, op: str = "experts",
+                weigh: Optional[bool] = None) -> None:
     """The experts' product over a plan: out[pos] = a[row(pos)] w[e(pos)]^T, or with w2 the
     gated pair.  w, w2: [E, N, K].  ``gather``: a's rows are tokens (row = the pair's token),
-    else sorted positions.  ``scatter``: out is [top * T, N] and a pair's row, times its
-    weight, goes to [choice * T + token]; else out's rows are sorted positions."""
+    else sorted positions.  ``scatter``: out is [top * T, N] and a pair's row goes to
+    [choice * T + token]; else out's rows are sorted positions.  ``weigh`` (default: with
+    ``scatter``): a row is multiplied by its pair's weight, on the gated pair before the
+    activation."""
     E, N, K = w.shape
     _dense(w, "w")
     assert a.stride(1) == 1 and out.stride(1) == 1 and a.shape[1] == K and out.shape[1] == N
@@ -387,9 +404,10 @@ def moe_grouped(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, plan: MoePl
         _check(library().agv_moe_grouped(
             _ptr(a), ctypes.c_longlong(a.stride(0)), _ptr(plan.tok) if gather else None,
             _ptr(plan.tok), _ptr(w), _ptr(w2), _ptr(out), ctypes.c_longlong(out.stride(0)),
-            _ptr(plan.dst) if scatter else None, _ptr(plan.wpos) if scatter else None,
+            _ptr(plan.dst) if scatter else None,
+            _ptr(plan.wpos) if (scatter if weigh is None else weigh) else None,
             _ptr(plan.tile_e), plan.tiles, plan.tile, N, K, dtype_code(a.dtype),
-            dtype_code(out.dtype), ACT[activation], _stream()))
+            dtype_code(out.dtype), *_act(activation, w2), _stream()))
 
 
 def moe_grouped_tc_supported(a: torch.Tensor, w: torch.Tensor) -> bool:
@@ -416,11 +434,12 @@ def moe_gather_rows(x: torch.Tensor, plan: MoePlan, xs: torch.Tensor) -> None:
 
 
 def moe_grouped_tc(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, plan: MoePlan,
-                   w2: Optional[torch.Tensor] = None, activation: str = "silu",
-                   scatter: bool = False, op: str = "experts") -> None:
+                   w2: Optional[torch.Tensor] = None, activation="silu",
+                   scatter: bool = False, op: str = "experts",
+                   weigh: Optional[bool] = None) -> None:
     """``moe_grouped`` in bfloat16 on the tensor cores; a's rows are sorted positions
     ([plan.rows, K]).  Gated: out [plan.rows, N] bfloat16.  Plain: out 32-bit, with
-    ``scatter`` [top * T, N] rows at [choice * T + token] times the pair's weight."""
+    ``scatter`` [top * T, N] rows at [choice * T + token]."""
     E, N, K = w.shape
     _dense(w, "w")
     assert a.shape == (plan.rows, K) and a.stride(1) == 1 and out.stride(1) == 1
@@ -437,8 +456,8 @@ def moe_grouped_tc(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, plan: Mo
         _check(library().agv_moe_grouped_tc(
             _ptr(a), ctypes.c_longlong(a.stride(0)), plan.rows, _ptr(plan.tok), _ptr(w), _ptr(w2),
             E, _ptr(out), ctypes.c_longlong(out.stride(0)), _ptr(plan.dst) if scatter else None,
-            _ptr(plan.wpos) if scatter else None, _ptr(plan.tile_e), plan.tiles, plan.tile, N, K,
-            ACT[activation], _stream()))
+            _ptr(plan.wpos) if (scatter if weigh is None else weigh) else None,
+            _ptr(plan.tile_e), plan.tiles, plan.tile, N, K, *_act(activation, w2), _stream()))
 
 
 def moe_tc_status() -> int:
@@ -459,7 +478,7 @@ def _linear_cost(x, w, w2, out):
 
 
 def linear_simt(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor,
-                w2: Optional[torch.Tensor] = None, activation: str = "gelu_tanh",
+                w2: Optional[torch.Tensor] = None, activation="gelu_tanh",
                 op: str = "linear") -> None:
     """out = x w^T, or act(x w^T) * (x w2^T); FFMA kernel (the 32-bit path)."""
     M, K = x.shape
@@ -476,7 +495,7 @@ def linear_simt(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor,
         _check(library().agv_linear_simt(
             _ptr(x), _ptr(w), _ptr(w2), _ptr(out), M, N, K, ctypes.c_longlong(x.stride(0)),
             ctypes.c_longlong(out.stride(0)), dtype_code(x.dtype), dtype_code(out.dtype),
-            ACT[activation], _stream()))
+            *_act(activation, w2), _stream()))
 
 
 # ------------------------------------------------------------------ attention
@@ -906,6 +925,71 @@ def delta_out(o: torch.Tensor, gate: torch.Tensor, w: torch.Tensor, eps: float, 
 
 
 
+HEAD_DELTA_COEF = 12        # numbers a token and head (checked against the library's)
+
+
+def head_delta_coef(u: torch.Tensor, decay: torch.Tensor, row: Optional[torch.Tensor],
+                    partial: Optional[torch.Tensor], W: int, b_offset: int, n_qk_heads: int,
+                    n_heads: int, head_dim: int, value_dim: int, unit_eps: float, q_mult: float,
+                    ctx, coef: torch.Tensor) -> None:
+    """What the delta rule with a decay per head needs of a token besides its vectors: u [T,
+    2 G d + H dv] = q | k | v after the convolution, decay [T, H, 2] (the decay first), beta =
+    sigmoid of columns ``b_offset`` .. + H of the stacked projection (32-bit rows [T, W] or
+    ``partial`` [S, T, W]); coef [T, H, 12], see ``csrc/delta_head.cu``."""
+    T = u.shape[0]
+    rp, ld, pp, ns = _f32_row_input(row, partial, T, W)
+    for t, n in ((u, "u"), (decay, "decay"), (coef, "coef")):
+        _f32(t, n); _dense(t, n)
+    assert u.shape == (T, 2 * n_qk_heads * head_dim + n_heads * value_dim)
+    assert decay.shape == (T, n_heads, 2)
+    lib = library()
+    assert coef.shape == (T, n_heads, lib.agv_head_delta_coef_numel())
+    with _span("delta_coef", T * 2 * n_qk_heads * head_dim * 4 + _nbytes(decay, coef)):
+        _check(lib.agv_head_delta_coef(
+            _ptr(u), _ptr(decay), rp, ld, pp, ns, T, W, b_offset, n_qk_heads, n_heads, head_dim,
+            value_dim, ctypes.c_float(unit_eps), ctypes.c_float(q_mult),
+            0 if ctx.mode == "decode" else 1, _ptr(ctx.seq_index), _ptr(ctx.cu_seqlens),
+            _ptr(coef), _stream()))
+
+
+def head_delta_scan(u: torch.Tensor, coef: torch.Tensor, out: torch.Tensor, ctx,
+                    state: torch.Tensor, n_qk_heads: int, n_heads: int, head_dim: int,
+                    value_dim: int) -> None:
+    """The recurrence  S <- g S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q  with one decay g
+    per head over the step's tokens, sequence by sequence; S [H, dv, d] of each sequence is read
+    from and written to ``state``.  All 32-bit; ``coef`` from ``head_delta_coef``."""
+    T = u.shape[0]
+    for t, n in ((u, "u"), (coef, "coef"), (out, "out")):
+        _f32(t, n); _dense(t, n)
+    assert u.shape == (T, 2 * n_qk_heads * head_dim + n_heads * value_dim)
+    assert out.shape == (T, n_heads * value_dim) and coef.shape[:2] == (T, n_heads)
+    sp, ss = _state_args(state)
+    with _span("delta_scan", _nbytes(u, coef, out) +
+               8 * ctx.batch * n_heads * head_dim * value_dim,
+               6 * T * n_heads * head_dim * value_dim):
+        _check(library().agv_head_delta_scan(
+            _ptr(u), _ptr(coef), _ptr(out), T, ctx.batch, n_qk_heads, n_heads, head_dim, value_dim,
+            0 if ctx.mode == "decode" else 1, sp, ss, _ptr(ctx.slots), _ptr(ctx.cu_seqlens),
+            _stream()))
+
+
+def head_delta_out(o: torch.Tensor, row: Optional[torch.Tensor], partial: Optional[torch.Tensor],
+                   W: int, g_offset: int, w: torch.Tensor, eps: float, n_heads: int,
+                   value_dim: int, silu: bool, ctx, y: torch.Tensor) -> None:
+    """y[t, h, :] = o[t, h, :] / rms(o[t, h, :]) * w * act(gate[t, h, :]), act silu or the
+    sigmoid; the gate is columns ``g_offset`` .. of the stacked projection; o is 32-bit [T, H *
+    dv], y is in the compute dtype."""
+    T = o.shape[0]
+    rp, ld, pp, ns = _f32_row_input(row, partial, T, W)
+    _f32(o, "o"); _f32(w, "w"); _dense(o, "o"); _dense(y, "y"); _dense(w, "w")
+    assert o.shape == y.shape == (T, n_heads * value_dim) and w.numel() == value_dim
+    with _span("delta_out", _nbytes(o, y) + T * n_heads * value_dim * 4 * max(ns, 1)):
+        _check(library().agv_head_delta_out(
+            _ptr(o), rp, ld, pp, ns, T, W, g_offset, _ptr(w), ctypes.c_float(eps), n_heads,
+            value_dim, 1 if silu else 0, _ptr(ctx.seq_index), _ptr(ctx.slots), _ptr(y),
+            dtype_code(y.dtype), _stream()))
+
+
 # ------------------------------------------------------- matrix memory (mLSTM)
 def mlstm_state_numel(n_heads: int, head_dim: int, value_dim: int) -> int:
     """32-bit values a sequence's matrix memory takes: S [H, d, dv], n [H, d] and the running
@@ -992,13 +1076,13 @@ def mlstm_out(num: torch.Tensor, den: torch.Tensor, den_eps: float, row: Optiona
 
 # ------------------------------------------------------- state-space mixers
 def ssm_conv(row: Optional[torch.Tensor], partial: Optional[torch.Tensor], T: int, W: int,
-             offset: int, taps: int, conv_w: torch.Tensor, conv_b: torch.Tensor,
+             offset: int, taps: int, conv_w: torch.Tensor, conv_b: Optional[torch.Tensor],
              out: torch.Tensor, rounded: Optional[torch.Tensor], state: torch.Tensor,
              state_off: int, ctx, dt_offset: int = 0, dt_bias: Optional[torch.Tensor] = None,
              neg_a: Optional[torch.Tensor] = None, coef: Optional[torch.Tensor] = None) -> None:
     """From channels ``offset`` .. of a token's row of the stacked projection (32-bit rows [T, W]
-    or ``partial`` [S, T, W]): a causal convolution over ``taps`` tokens per channel with a bias,
-    then silu, into out [T, C] (32-bit) and, if given, ``rounded`` [T, C] (another dtype).
+    or ``partial`` [S, T, W]): a causal convolution over ``taps`` tokens per channel with a bias
+    (None: without), then silu, into out [T, C] (32-bit) and, if given, ``rounded`` [T, C] (another dtype).
     Earlier inputs come from the step's rows or from the ring in ``state`` at ``state_off``,
     which is brought up to date.  With ``coef`` [T, H, 2]: the columns ``dt_offset`` .. + H are
     step sizes, dt = softplus(x + dt_bias), and coef receives (exp(neg_a * dt), dt)."""
@@ -1009,7 +1093,8 @@ def ssm_conv(row: Optional[torch.Tensor], partial: Optional[torch.Tensor], T: in
         _f32(t, n)
         if t is not None:
             _dense(t, n)
-    assert conv_w.shape == (C, taps) and conv_b.numel() == C and out.shape == (T, C)
+    assert conv_w.shape == (C, taps) and (conv_b is None or conv_b.numel() == C)
+    assert out.shape == (T, C)
     n_dt = 0
     if coef is not None:
         n_dt = dt_bias.numel()
@@ -1134,8 +1219,8 @@ def gated_join(h: Optional[torch.Tensor], terms, gate_row: Optional[torch.Tensor
     h += sum_i mult_i * sigmoid(logits[gate_i] + bias[gate_i]) * y_i, then x = rmsnorm(h) * w_next
     if there is one (x alone: the sum as it is; h None: the sum starts at zero).
 
-    ``terms``: (y, mult, gate) with y [R, H] or 32-bit partial sums [S, R, H] and gate the index
-    of its gate or -1; the gates' logits are stacked, 32-bit [R, G * H] or [S, R, G * H]."""
+    ``terms``: (y, mult, gate) with y [R, H], 32-bit partial sums [S, R, H] or one row [H] that
+    every row takes (a bias; not the first term), and gate the index of its gate or -1; the gates' logits are stacked, 32-bit [R, G * H] or [S, R, G * H]."""
     first = terms[0][0]
     R, H = first.shape[-2:]
     n = len(terms)
@@ -1143,11 +1228,11 @@ def gated_join(h: Optional[torch.Tensor], terms, gate_row: Optional[torch.Tensor
     mults, gates = (ctypes.c_float * n)(), (ctypes.c_int * n)()
     for i, (y, mult, gate) in enumerate(terms):
         _dense(y, "y")
-        assert y.shape[-2:] == (R, H)
+        assert y.shape[-2:] == (R, H) or y.shape == (H,)
         if y.dim() == 3:
             _f32(y, "y")
         ys[i], dts[i] = _ptr(y), dtype_code(y.dtype)
-        splits[i] = y.shape[0] if y.dim() == 3 else 1
+        splits[i] = y.shape[0] if y.dim() == 3 else 1 if y.dim() == 2 else 0
         mults[i], gates[i] = float(mult), int(gate)
     n_gates = 0
     rp, ld = ctypes.c_void_p(0), ctypes.c_longlong(0)
@@ -1295,7 +1380,7 @@ def sample(logits: torch.Tensor, out: torch.Tensor, temperature: float, top_k: i
 
 
 def linear_tc(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor,
-              w2: Optional[torch.Tensor] = None, activation: str = "gelu_tanh",
+              w2: Optional[torch.Tensor] = None, activation="gelu_tanh",
               splits: int = 1, token_tile: int = 0, cluster: int = 0,
               op: str = "linear") -> None:
     """bfloat16 product on the tensor cores (tcgen05 + TMA).
@@ -1325,7 +1410,7 @@ def linear_tc(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor,
     with _span(op, *_linear_cost(x, w, w2, out)):
         _check(library().agv_linear_tc(
             _ptr(x), _ptr(w), _ptr(w2), _ptr(out), T, N, K, ctypes.c_longlong(x.stride(0)),
-            ctypes.c_longlong(ldc), dtype_code(out.dtype), ACT[activation], splits, cluster,
+            ctypes.c_longlong(ldc), dtype_code(out.dtype), *_act(activation, w2), splits, cluster,
             token_tile, _stream()))
 
 
@@ -1397,7 +1482,7 @@ def n_sms() -> int:
 _PREFILL_TC = os.environ.get("AGAVE_B200_PREFILL_ATTENTION", "tcgen05") != "mma"
 
 def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor,
-           w2: Optional[torch.Tensor] = None, activation: str = "gelu_tanh",
+           w2: Optional[torch.Tensor] = None, activation="gelu_tanh",
            op: str = "linear") -> None:
     """out = x w^T (or the gated pair).  Which kernel runs follows from the dtype and the
     weight's shape; how K is cut into ranges (and with it the order of the 32-bit sums)

@@ -5,5 +5,6 @@ from . import zazerax as _zazerax    # registers the architecture
 from . import bovozen as _bovozen    # registers the architecture
 from . import kadavik as _kadavik    # registers the architecture
 from . import savovik as _savovik    # registers the architecture
+from . import pubunex as _pubunex    # registers the architecture
 
 __all__ = ["DecoderModel", "decoder_param_specs"]

@@ -249,17 +249,33 @@ class DecoderModel:
         sched = spec.schedule
         if not sched:
             return h
+        start = None                       # the stream before the first block, where it is needed again
+        if any(c.add_embedding for c in sched):
+            start = ctx.new(T, spec.hidden_size, dtype=torch.float32)
+            start.copy_(h)
         if self._few_tokens(ctx):
             return self._blocks_few_tokens(h, ctx)
         x = ctx.new(T, spec.hidden_size)
-        self.blocks[sched[0].block].entry_norm.forward(h, x)
+        if sched[0].add_embedding:
+            self.blocks[sched[0].block].entry_norm.after_residual(h, start, x)
+        else:
+            self.blocks[sched[0].block].entry_norm.forward(h, x)
         for i, call in enumerate(sched):
             if ctx.cancel is not None and ctx.cancel.is_set():
                 raise Cancelled(f"cancelled before block {i} of {len(sched)}")
             nxt = self.blocks[sched[i + 1].block].entry_norm if i + 1 < len(sched) else None
             st = getattr(call, "state", None)
             ctx.state_entry = call.cache if st is None else st
-            x = self.blocks[call.block].forward(h, x, ctx, call.cache, call.writes_cache, nxt)
+            block = self.blocks[call.block]
+            again = nxt is not None and sched[i + 1].add_embedding
+            if not again or getattr(block, "joins_extra", False):
+                ctx.join_extra = start if again else None
+                x = block.forward(h, x, ctx, call.cache, call.writes_cache, nxt)
+                ctx.join_extra = None
+            else:
+                block.forward(h, x, ctx, call.cache, call.writes_cache, None)
+                x = ctx.new(T, spec.hidden_size)
+                nxt.after_residual(h, start, x)
         return h
 
     def logits(self, h: torch.Tensor, rows: torch.Tensor, ctx,

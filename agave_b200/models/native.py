@@ -68,14 +68,15 @@ def standard_blocks(model) -> bool:
     function and the few-token decode path know how to run."""
     if model.head is None or model.stream_position is not None:
         return False
-    if any(not c.writes_cache for c in model.spec.schedule):
+    if any(not c.writes_cache or c.add_embedding for c in model.spec.schedule):
         return False
     for b in model.blocks:
         if type(b) is not Block or type(b.mixer) is not AttentionMixer or \
                 type(b.ffn) is not GatedFeedForward:
             return False
         if not isinstance(b.mixer.spec, AttentionSpec) or \
-                not isinstance(b.ffn.spec, GatedFeedForwardSpec):
+                not isinstance(b.ffn.spec, GatedFeedForwardSpec) or \
+                not isinstance(b.ffn.gate_up.activation, str):
             return False
         for n in (b.pre_mixer_norm, b.pre_ffn_norm, b.post_mixer_norm, b.post_ffn_norm):
             if n is not None and type(n) is not RMSNorm:

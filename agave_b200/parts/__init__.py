@@ -6,7 +6,7 @@ from .norm import Identity, LayerNorm, RMSNorm
 from .rope import RotaryEmbedding
 from .attention import AttentionMixer
 from .latent import LatentAttentionMixer
-from .delta import ChannelDeltaMixer
+from .delta import ChannelDeltaMixer, HeadDeltaMixer
 from .position import LearnedPosition
 from .feedforward import DenseFeedForward, GatedFeedForward
 from .moe import RoutedFeedForward
@@ -20,6 +20,6 @@ __all__ = ["KVRequest", "ParamSpec", "StateRequest", "feed_forward_class", "mixe
            "register_block", "register_feed_forward", "register_mixer", "register_norm",
            "register_position", "register_stream_position", "RMSNorm", "LayerNorm",
            "RoutedFeedForward", "RotaryEmbedding", "Identity", "LatentAttentionMixer",
-           "DenseFeedForward", "ChannelDeltaMixer", "LearnedPosition",
+           "DenseFeedForward", "ChannelDeltaMixer", "HeadDeltaMixer", "LearnedPosition",
            "SelectiveScanMixer", "StateSpaceMixer", "ParallelBlock", "SideBySideMixer",
            "AttentionMixer", "GatedFeedForward", "Block", "GatedLinear", "Linear"]

@@ -42,8 +42,9 @@ the cache for keys and values *and* for state); and an output gate sigmoid(W_g x
 concatenated heads (``out_gate``; tensor ``g_proj.weight``, stacked under q | k | v); biases on
 the q, k and v projections (``qkv_bias``; tensors ``q_proj.bias`` ...); neighbouring dimensions
 rotated as pairs (the position part's ``interleaved``); every value head divided by its root
-mean square before it is cached (``value_norm_eps``); and a soft cap on the scaled scores
-(``softcap``).
+mean square before it is cached (``value_norm_eps``); a soft cap on the scaled scores
+(``softcap``); and a bias on the output projection (``out_bias``; tensor ``o_proj.bias``), which
+a block that joins the branches itself takes as a term of that sum.
 """
 from __future__ import annotations
 
@@ -93,6 +94,8 @@ class AttentionMixer:
         self.softcap = float(getattr(spec, "softcap", None) or 0.0)
         self.qkv_bias = bool(getattr(spec, "qkv_bias", False))
         self.bias: Optional[torch.Tensor] = None
+        self.has_out_bias = bool(getattr(spec, "out_bias", False))
+        self.out_bias: Optional[torch.Tensor] = None
         veps = getattr(spec, "value_norm_eps", None)
         self.value_eps = None if veps is None else float(veps)
         self.interleaved = bool(self.position is not None and
@@ -133,7 +136,7 @@ class AttentionMixer:
                       and self.slope_spec is None and self.chunk is None
                       and self.value_mix is None and not self.keep_first
                       and not self.conv_taps and not self.out_gate
-                      and not self.row_extras and not self.softcap)
+                      and not self.row_extras and not self.softcap and not self.has_out_bias)
 
     @classmethod
     def param_specs(cls, spec: AttentionSpec, hidden_size: int) -> Dict[str, ParamSpec]:
@@ -173,6 +176,8 @@ class AttentionMixer:
             if own_kv:
                 p["k_proj.bias"] = ParamSpec((kv,), "float32")
                 p["v_proj.bias"] = ParamSpec((spec.n_kv_heads * vd,), "float32")
+        if getattr(spec, "out_bias", False):
+            p["o_proj.bias"] = ParamSpec((hidden_size,), "float32")
         return p
 
     @staticmethod
@@ -242,6 +247,9 @@ class AttentionMixer:
             self.bias = torch.cat([tensors[n].to(device=device, dtype=torch.float32)
                                    for n in names]).contiguous()
         self.out = Linear(mat("o_proj.weight").contiguous(), role="out_proj")
+        if self.has_out_bias:
+            self.out_bias = tensors["o_proj.bias"].to(device=device,
+                                                      dtype=torch.float32).contiguous()
         if self.spec.qk_norm is not None:
             add = 1.0 if self.spec.qk_norm.zero_centered else 0.0
             self.q_norm_weight = (tensors["q_norm.weight"].to(device=device, dtype=torch.float32)
@@ -278,7 +286,22 @@ class AttentionMixer:
         if self.value_mix is not None and self.value_mix.source is not None:
             self.mix_weight = float(tensors["value_mix"].to(torch.float32).reshape(()).item())
 
+    def forward_terms(self, x: torch.Tensor, ctx, cache_entry: int, writes_cache: bool):
+        """The branch as terms of a sum with their multipliers, for a block that joins them
+        itself: the output product and, where there is one, its bias (one row for all)."""
+        y = self._branch(x, ctx, cache_entry, writes_cache)
+        return [(y, 1.0)] + ([(self.out_bias, 1.0)] if self.out_bias is not None else [])
+
     def forward(self, x: torch.Tensor, ctx, cache_entry: int, writes_cache: bool) -> torch.Tensor:
+        terms = self.forward_terms(x, ctx, cache_entry, writes_cache)
+        if len(terms) == 1:
+            return terms[0][0]
+        y = ctx.new(x.shape[0], self.hidden_size, dtype=torch.float32)
+        kernels.gated_join(None, [(t, m, -1) for t, m in terms], None, None, None, None, 0.0, y)
+        return y.unsqueeze(0)
+
+    def _branch(self, x: torch.Tensor, ctx, cache_entry: int, writes_cache: bool) -> torch.Tensor:
+        """The output product without its bias."""
         if self.conv_taps or self.out_gate:
             return self._forward_conv(x, ctx, cache_entry, writes_cache)
         if not self.plain:

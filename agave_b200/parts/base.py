@@ -95,7 +95,9 @@ def register_block(kind: str, cls: type) -> None:
     ``cache_request()`` and
     ``forward(h, x, ctx, cache_entry, writes_cache, next_norm) -> x_next``: h is the
     32-bit stream [T, H], updated in place; x = entry_norm(h); x_next = next_norm(h)
-    after the update, or None when next_norm is None."""
+    after the update, or None when next_norm is None.  A class with ``joins_extra`` True adds
+    ``ctx.join_extra`` ([T, H] 32-bit, or None) to the stream after its branches; for others the
+    decoder does that in a launch of its own."""
     _BLOCKS[kind] = cls
 
 

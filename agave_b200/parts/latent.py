@@ -9,7 +9,8 @@ A heads, d = ``head_dim`` unrotated and r = ``rot_dim`` rotated query/key dimens
 
 and the concatenated heads, times sigmoid(W_g x) (element by element, or one value per head),
 go through W_o.  The queries come from x directly (W_q) or, with ``q_rank``, through a normed
-latent of their own (W_uq rmsnorm(W_dq x)).
+latent of their own (W_uq rmsnorm(W_dq x)).  ``sink``: a learned logit per head joins the
+softmax denominator once, in prompts and while decoding.
 
 Two ways to compute the same sums.  A prompt step rebuilds keys and values for its tokens
 (the products W_uk c and W_uv c) and runs ordinary multi-head attention over the step's own
@@ -56,6 +57,7 @@ class LatentAttentionMixer:
         self.v_up: Optional[torch.Tensor] = None       # [A, value_dim, kv_rank]
         self.out: Optional[Linear] = None
         self.w_q_norm = self.w_c_norm = None
+        self.sinks: Optional[torch.Tensor] = None
 
     @classmethod
     def param_specs(cls, spec: LatentAttentionSpec, hidden_size: int) -> Dict[str, ParamSpec]:
@@ -75,6 +77,8 @@ class LatentAttentionMixer:
             p["gate.weight"] = ParamSpec((A * dv, hidden_size))
         elif spec.gate == "head":
             p["gate.weight"] = ParamSpec((A, hidden_size))
+        if spec.sink:
+            p["sink"] = ParamSpec((A,), "float32")
         p["o_proj.weight"] = ParamSpec((hidden_size, A * dv))
         return p
 
@@ -106,6 +110,8 @@ class LatentAttentionMixer:
         self.k_absorb = uk.view(A, d, R).transpose(1, 2).contiguous()
         self.v_up = uv.view(A, dv, R).contiguous()
         self.out = Linear(mat("o_proj.weight").contiguous(), role="out_proj")
+        if s.sink:
+            self.sinks = tensors["sink"].to(device=device, dtype=torch.float32).contiguous()
         if hasattr(self.position, "prepare"):
             self.position.prepare(device)
 
@@ -135,7 +141,7 @@ class LatentAttentionMixer:
             k = ctx.new(T, A * hw)
             kernels.assemble_keys(self.k_up(c), kr, k, A, d, r)
             kernels.attention_prefill(q, k, self.v_up_prompt(c), out, ctx, A, A, hw, s.scale, 0,
-                                      value_dim=dv, op="latent_attention")
+                                      value_dim=dv, sinks=self.sinks, op="latent_attention")
         else:
             # the key up-projection goes into the query (the rotated part passes through);
             # the heads attend to the cache rows themselves
@@ -147,13 +153,13 @@ class LatentAttentionMixer:
                 # head in its group; the r values behind the latent's weighted sum are unused
                 lat = ctx.new(T, A, D)
                 kernels.attention_decode(ql.view(T, A * D), lat.view(T, A * D), view, ctx, A, 1, D,
-                                         s.scale, 0, op="latent_attention")
+                                         s.scale, 0, sinks=self.sinks, op="latent_attention")
                 lat = lat[:, :, :R]
             else:
                 lat = ctx.new(T, A, R)
                 kernels.attention_decode(ql.view(T, A * D), lat.view(T, A * R), view, ctx, A, 1, D,
                                          s.scale, 0, value_dim=R, values_in_keys=True,
-                                         op="latent_attention")
+                                         sinks=self.sinks, op="latent_attention")
             # (the output gate rides on the value up-projection)
             kernels.heads_linear(lat, self.v_up, out.view(T, A, dv), op="v_up",
                                  gate=row[:, Q + R + r:] if G else None)

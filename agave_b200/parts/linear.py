@@ -14,6 +14,7 @@ from typing import Optional
 import torch
 
 from .. import kernels
+from ..config.base import ClampedGateSpec
 
 
 class Linear:
@@ -45,13 +46,24 @@ class Linear:
         return kernels.linear_partial(x, self.weight, cheap_sum, op=self.role)
 
 
-class GatedLinear:
-    """act(x wg^T) * (x wu^T) in one kernel."""
+def gate_activation(activation):
+    """A gated pair's activation as the kernels take it: a name, or from a ``ClampedGateSpec``
+    ("clamped", alpha, limit)."""
+    if isinstance(activation, ClampedGateSpec):
+        if not activation.limit > 0:
+            raise ValueError("the limit of a clamped gate must be positive")
+        return ("clamped", float(activation.alpha), float(activation.limit))
+    return activation
 
-    def __init__(self, w_gate: torch.Tensor, w_up: torch.Tensor, activation: str,
+
+class GatedLinear:
+    """act(x wg^T) * (x wu^T), or another function of the two, in one kernel."""
+
+    def __init__(self, w_gate: torch.Tensor, w_up: torch.Tensor, activation,
                  role: str = "gate_up"):
         assert w_gate.shape == w_up.shape
-        self.w_gate, self.w_up, self.activation, self.role = w_gate, w_up, activation, role
+        self.w_gate, self.w_up, self.role = w_gate, w_up, role
+        self.activation = gate_activation(activation)
         self.out_features, self.in_features = w_gate.shape
 
     def __call__(self, x: torch.Tensor, out: Optional[torch.Tensor] = None) -> torch.Tensor:

@@ -26,7 +26,11 @@ slice of the partial sums; scores that are the softmax over all the router's out
 chosen ones renormalised and multiplied by a constant (``weighting`` "softmax_all",
 ``route_scale``); and identity experts (``n_identity``): router outputs beyond the experts
 that have no tensors and whose output is the input itself, times the weight.  A pair that
-chose one is left out of the plan, and a small kernel writes its row of the partial sums.
+chose one is left out of the plan, and a small kernel writes its row of the partial sums; a
+weight that multiplies the expert's input (``weigh_input``: expert(w x); the gate/up product's
+epilogue multiplies its two 32-bit sums by it, so w x is never rounded); a shared expert
+without a gate (``shared_gate`` False) or with an activation of its own
+(``shared_activation``).
 """
 from __future__ import annotations
 
@@ -37,7 +41,7 @@ import torch
 from .. import kernels
 from ..config.base import RoutedFeedForwardSpec
 from .base import ParamSpec, register_feed_forward
-from .linear import GatedLinear, Linear
+from .linear import GatedLinear, Linear, gate_activation
 
 
 class RoutedFeedForward:
@@ -62,6 +66,12 @@ class RoutedFeedForward:
             raise ValueError("weights by softmax over the chosen logits go without a correction")
         self.has_bias = bool(getattr(spec, "router_bias", False))
         self.shared_size = int(getattr(spec, "shared_size", 0) or 0)
+        self.has_shared_gate = bool(getattr(spec, "shared_gate", True))
+        self.activation = gate_activation(spec.activation)
+        self.shared_activation = getattr(spec, "shared_activation", None) or spec.activation
+        self.weigh_input = bool(getattr(spec, "weigh_input", False))
+        if self.weigh_input and self.n_identity:
+            raise ValueError("a weight on the experts' input goes without identity experts")
         self.router_bias: Optional[torch.Tensor] = None
         self.shared_gate_up = self.shared_down = self.shared_gate = None
         self.w_router: Optional[torch.Tensor] = None
@@ -86,7 +96,8 @@ class RoutedFeedForward:
             p["shared.gate_proj.weight"] = ParamSpec((sf, hidden_size))
             p["shared.up_proj.weight"] = ParamSpec((sf, hidden_size))
             p["shared.down_proj.weight"] = ParamSpec((hidden_size, sf))
-            p["shared.gate.weight"] = ParamSpec((1, hidden_size))
+            if getattr(spec, "shared_gate", True):
+                p["shared.gate.weight"] = ParamSpec((1, hidden_size))
         return p
 
     def load(self, tensors: Dict[str, torch.Tensor], dtype: torch.dtype,
@@ -106,10 +117,11 @@ class RoutedFeedForward:
             def mat(name):
                 return tensors[name].to(device=device, dtype=dtype).contiguous()
             self.shared_gate_up = GatedLinear(mat("shared.gate_proj.weight"),
-                                              mat("shared.up_proj.weight"), self.spec.activation,
+                                              mat("shared.up_proj.weight"), self.shared_activation,
                                               role="shared_gate_up")
             self.shared_down = Linear(mat("shared.down_proj.weight"), role="shared_down")
-            self.shared_gate = mat("shared.gate.weight").reshape(-1).contiguous()
+            if self.has_shared_gate:
+                self.shared_gate = mat("shared.gate.weight").reshape(-1).contiguous()
 
     def route(self, x: torch.Tensor):
         """(ids [T, top] int32, weights [T, top] 32-bit) of the tokens of x."""
@@ -126,7 +138,8 @@ class RoutedFeedForward:
     def _shared(self, x: torch.Tensor, out: torch.Tensor) -> None:
         """out [T, H] (32-bit) = sigmoid(w_sg . x) * down(act(gate x) * up x)."""
         self.shared_down(self.shared_gate_up(x), out=out)
-        kernels.row_gate(x, self.shared_gate, out)
+        if self.has_shared_gate:
+            kernels.row_gate(x, self.shared_gate, out)
 
     def forward(self, x: torch.Tensor, ctx) -> torch.Tensor:
         s = self.spec
@@ -147,14 +160,15 @@ class RoutedFeedForward:
             xs = torch.empty((plan.rows, H), dtype=x.dtype, device=x.device)
             kernels.moe_gather_rows(x, plan, xs)
             kernels.moe_grouped_tc(xs, self.w_gate, z, plan, w2=self.w_up,
-                                   activation=s.activation, op="experts_gate_up")
+                                   activation=self.activation, weigh=self.weigh_input,
+                                   op="experts_gate_up")
             kernels.moe_grouped_tc(z, self.w_down, y[:s.top].view(s.top * T, H), plan, scatter=True,
-                                   op="experts_down")
+                                   weigh=not self.weigh_input, op="experts_down")
             return y
-        kernels.moe_grouped(x, self.w_gate, z, plan, w2=self.w_up, activation=s.activation,
-                            gather=True, op="experts_gate_up")
+        kernels.moe_grouped(x, self.w_gate, z, plan, w2=self.w_up, activation=self.activation,
+                            gather=True, weigh=self.weigh_input, op="experts_gate_up")
         kernels.moe_grouped(z, self.w_down, y[:s.top].view(s.top * T, H), plan, scatter=True,
-                            op="experts_down")
+                            weigh=not self.weigh_input, op="experts_down")
         return y
 
 

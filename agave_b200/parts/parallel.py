@@ -10,8 +10,9 @@ and values and at most one a fixed-size state.
     h += sigmoid(W_m x + b_m) * mixer(x) + sigmoid(W_f x + b_f) * ffn(x)
 
 element by element, or without the gates.  The two gates' projections are one stacked product;
-the gates, the branches' sums over ranges of K, the scales of mixers side by side, the residual
-sum and the norm that feeds the next block are one launch.
+the gates, the branches' sums over ranges of K, the scales of mixers side by side, the bias of a
+mixer's output product, what the run order adds to the stream after the block, the residual sum
+and the norm that feeds the next block are one launch.
 """
 from __future__ import annotations
 
@@ -114,6 +115,9 @@ class ParallelBlock:
                 out[f"{name}.bias"] = ParamSpec((hidden_size,), "float32")
         return out
 
+    # the block adds ``ctx.join_extra`` (a 32-bit [T, H] or None) to the stream in its own join
+    joins_extra = True
+
     @property
     def entry_norm(self):
         return self.norm
@@ -149,6 +153,9 @@ class ParallelBlock:
         terms = [(y, m, 0 if self.gated else -1) for y, m in branches]
         if self.ffn is not None:
             terms.append((self.ffn.forward(x, ctx), 1.0, 1 if self.gated else -1))
+        extra = getattr(ctx, "join_extra", None)
+        if extra is not None:
+            terms.append((extra, 1.0, -1))
         row = part = None
         if self.gated:
             row, part = project_f32(self.gates, x)
