@@ -22,7 +22,7 @@
 // the same sums with S as it was before the round, so a round has one pass of dot products with
 // the state, whose reductions over a column's lanes do not wait for one another.  What does not
 // depend on the state (the dot products among a round's k and q, the decays' products, all of it
-// folded into twelve numbers a token and head) is made by a launch before for all rounds at
+// folded into a few numbers a token and head) is made by a launch before for all rounds at
 // once; the vectors themselves stay as the convolution left them.  A round begins at the first
 // token a sequence brings in the step; a decode step's rounds are one token.
 //
@@ -32,9 +32,11 @@
 
 namespace {
 
-constexpr int DH_R = 16;           // rows of a column a lane holds
-constexpr int DH_ROUND = 4;        // tokens a round of a prompt
-constexpr int DH_COEF = 12;        // numbers a token and head
+// tokens a round of a prompt, by the size of a key head
+__host__ __device__ constexpr int head_round(int d) { return d > 32 ? 8 : 4; }
+constexpr int DH_MAX_D = 512;
+// numbers a token and head, whole quads
+__host__ __device__ constexpr int head_coefs(int n) { return (4 + 2 * n + 3) / 4 * 4; }
 
 struct HeadDims {
     int G, H, d, dv;
@@ -46,30 +48,46 @@ __device__ __forceinline__ float silu_f(float t) { return t / (1.0f + expf(-t));
 __device__ __forceinline__ float sigmoid_f(float t) { return 1.0f / (1.0f + expf(-t)); }
 
 // ------------------------------------------------------------- coefficients
-// A warp per (token, query/key head); the first token of a round works for the whole round.
-// Layout of a token's numbers (i its place in the round, n the round's last place):
-//   0 beta   1 beta G_i0 r_i   2..4 beta G_ij r_i r_j (k_i . k_j), j = 0..2
-//   5 G_i0 s_i   6..9 G_ij s_i r_j (q_i . k_j), j = 0..3   10 G_nj r_j with j = i   11 G_n0
-// (zeros where j >= i, or j > i).
+// A warp per (round, query/key head): the dot products by lanes over d, folded so that every lane ends with a few finished sums, then a
+// lane per (head, token).  Layout of a token's numbers (i its place in the round, n the round's
+// last place):
+//   0 beta   1 beta G_i0 r_i   2 G_i0 s_i   3 G_ni r_i
+//   4 + j: beta G_ij r_i r_j (k_i . k_j) for j < i, else 0; the last of them is G_n0 instead
+//   4 + N + j: G_ij s_i r_j (q_i . k_j) for j <= i, else 0
+//
+// Sequence b has the rounds from number cu[b] / N + b on: room for its own, ceil(len / N), and
+// T / N + B in all (a number that is no sequence's round has nothing to do).
+constexpr int DH_COEF_WARPS = 8;
+
 template <int N>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(DH_COEF_WARPS * 32)
 delta_coef_kernel(const float* __restrict__ u, const float* __restrict__ decay, RowIn<float> in,
-                  int b_off, HeadDims dm, int n_tokens, float eps_unit, float q_mult,
-                  const int* __restrict__ seq_index, const int* __restrict__ cu,
-                  float* __restrict__ coef) {
+                  int b_off, HeadDims dm, int n_tokens, int B, float eps_unit, float q_mult,
+                  const int* __restrict__ cu, float* __restrict__ coef) {
     pdl_wait();
     pdl_launch_next();
-    const int lane = threadIdx.x & 31;
-    const long long w = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
-    if (w >= (long long)n_tokens * dm.G) return;
-    const int t = (int)(w / dm.G), grp = (int)(w - (long long)t * dm.G);
-    const int b = seq_index[t], first = cu[b], end = cu[b + 1];
-    if (N > 1 && (t - first) % N != 0) return;
+    constexpr int TRI = N * (N + 1) / 2, SUMS = N + 2 * TRI, M = (SUMS + 31) / 32 * 32;
+    __shared__ float sums[DH_COEF_WARPS][M];       // |q_i|^2, k_i . k_j, q_i . k_j (j <= i)
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const long long w = (long long)blockIdx.x * DH_COEF_WARPS + warp;
+    const int round = (int)(w / dm.G), grp = (int)(w - (long long)round * dm.G);
+    if (round >= n_tokens / N + B) return;
+    int b = 0;                                     // the last sequence that starts at or before it
+    for (int hi = B - 1; b < hi;) {
+        const int mid = (b + hi + 1) >> 1;
+        if (cu[mid] / N + mid <= round) b = mid;
+        else hi = mid - 1;
+    }
+    const int first = cu[b], end = cu[b + 1];
+    const int t = first + (round - (first / N + b)) * N;
+    if (t >= end) return;
     const int m = min(N, end - t);
     const int C = dm.C(), d = dm.d;
     const float* q0 = u + (size_t)t * C + (size_t)grp * d;
     const float* k0 = q0 + dm.nq();
-    float qq[N] = {}, kk[N][N] = {}, qk[N][N] = {};
+    float v[M];
+#pragma unroll
+    for (int x = 0; x < M; ++x) v[x] = 0.f;
 #pragma unroll 2
     for (int r = lane; r < d; r += 32) {
         float q[N], k[N];
@@ -80,66 +98,68 @@ delta_coef_kernel(const float* __restrict__ u, const float* __restrict__ decay, 
         }
 #pragma unroll
         for (int i = 0; i < N; ++i) {
-            qq[i] = fmaf(q[i], q[i], qq[i]);
+            v[i] = fmaf(q[i], q[i], v[i]);
 #pragma unroll
             for (int j = 0; j <= i; ++j) {
-                kk[i][j] = fmaf(k[i], k[j], kk[i][j]);
-                qk[i][j] = fmaf(q[i], k[j], qk[i][j]);
+                const int x = N + i * (i + 1) / 2 + j;
+                v[x] = fmaf(k[i], k[j], v[x]);
+                v[x + TRI] = fmaf(q[i], k[j], v[x + TRI]);
             }
         }
     }
+    int at = 0;
 #pragma unroll
-    for (int i = 0; i < N; ++i) {
-        qq[i] = warp_sum(qq[i]);
+    for (int bit = 16, half = M / 2; bit >= 1; bit >>= 1, half >>= 1) {
+        const bool up = lane & bit;
+        if (up) at += half;
 #pragma unroll
-        for (int j = 0; j <= i; ++j) {
-            kk[i][j] = warp_sum(kk[i][j]);
-            qk[i][j] = warp_sum(qk[i][j]);
+        for (int x = 0; x < half; ++x) {
+            const float out = up ? v[x] : v[x + half], keep = up ? v[x + half] : v[x];
+            v[x] = keep + __shfl_xor_sync(0xffffffffu, out, bit);
         }
     }
-    float rk[N], rq[N];
 #pragma unroll
-    for (int i = 0; i < N; ++i) {
-        rk[i] = 1.0f / sqrtf(kk[i][i] + eps_unit);
-        rq[i] = q_mult / sqrtf(qq[i] + eps_unit);
-    }
+    for (int x = 0; x < M / 32; ++x) sums[warp][at + x] = v[x];
+    __syncwarp();
+    const float* qq = sums[warp];
+    const float* kk = qq + N;
+    const float* qk = kk + TRI;
     const int per = dm.H / dm.G;
-    for (int hh = lane; hh < per; hh += 32) {
-        const int h = grp * per + hh;
+    for (int e = lane; e < per * N; e += 32) {
+        const int i = e % N, h = grp * per + e / N;
+        if (i >= m) continue;
         float g[N];
 #pragma unroll
-        for (int i = 0; i < N; ++i)
-            g[i] = i < m ? decay[((size_t)(t + i) * dm.H + h) * 2] : 1.f;
-        float total = 1.f;
+        for (int j = 0; j < N; ++j) g[j] = j < m ? decay[((size_t)(t + j) * dm.H + h) * 2] : 1.f;
+        const float beta = sigmoid_f(in.at(t + i, b_off + h));
+        const int tri = i * (i + 1) / 2;
+        const float ri = 1.0f / sqrtf(kk[tri + i] + eps_unit), si = q_mult / sqrtf(qq[i] + eps_unit);
+        float before = 1.f, after = 1.f;                     // g_1 .. g_i, g_(i+1) .. g_n
 #pragma unroll
-        for (int i = 0; i < N; ++i) total *= g[i];
-        float from_start = 1.f;
-#pragma unroll
-        for (int i = 0; i < N; ++i) {
-            if (i >= m) break;
-            from_start *= g[i];
-            const float beta = sigmoid_f(in.at(t + i, b_off + h));
-            float c[DH_COEF] = {};
-            c[0] = beta;
-            c[1] = beta * from_start * rk[i];
-            c[5] = from_start * rq[i];
-            float between = 1.f;                             // g_(j+1) .. g_i
-#pragma unroll
-            for (int j = i; j >= 0; --j) {
-                if (j < i) c[2 + j] = beta * between * rk[i] * rk[j] * kk[i][j];
-                c[6 + j] = between * rq[i] * rk[j] * qk[i][j];
-                between *= g[j];
-            }
-            float after = 1.f;                               // g_(i+1) .. g_n
-#pragma unroll
-            for (int j = i + 1; j < N; ++j) after *= g[j];
-            c[10] = after * rk[i];
-            c[11] = total;
-            float4* o = reinterpret_cast<float4*>(coef + ((size_t)(t + i) * dm.H + h) * DH_COEF);
-            o[0] = make_float4(c[0], c[1], c[2], c[3]);
-            o[1] = make_float4(c[4], c[5], c[6], c[7]);
-            o[2] = make_float4(c[8], c[9], c[10], c[11]);
+        for (int j = 0; j < N; ++j) {
+            if (j <= i) before *= g[j];
+            else after *= g[j];
         }
+        constexpr int NF = head_coefs(N);
+        float c[NF] = {};
+        c[0] = beta;
+        c[1] = beta * before * ri;
+        c[2] = before * si;
+        c[3] = after * ri;
+        float between = 1.f;                                 // g_(j+1) .. g_i
+#pragma unroll
+        for (int j = N - 1; j >= 0; --j) {
+            if (j > i) continue;
+            const float rj = 1.0f / sqrtf(kk[j * (j + 1) / 2 + j] + eps_unit);
+            if (j < i) c[4 + j] = beta * between * ri * rj * kk[tri + j];
+            c[4 + N + j] = between * si * rj * qk[tri + j];
+            between *= g[j];
+        }
+        c[4 + N - 1] = before * after;
+        float4* o = reinterpret_cast<float4*>(coef + ((size_t)(t + i) * dm.H + h) * NF);
+#pragma unroll
+        for (int x = 0; x < NF / 4; ++x)
+            o[x] = make_float4(c[4 * x], c[4 * x + 1], c[4 * x + 2], c[4 * x + 3]);
     }
 }
 
@@ -158,7 +178,7 @@ __device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_gr
 
 struct HeadScanArgs {
     const float* u;            // [T, C]: q | k | v after the convolution
-    const float* coef;         // [T, H, 12]
+    const float* coef;         // [T, H, head_coefs(tokens a round)]
     float* out;                // [T, H * dv]
     float* state;              // [n_slots, stride]: S [H, dv, d] at 0
     long long stride;
@@ -170,19 +190,25 @@ struct HeadScanArgs {
     int vec_s;                 // a column of S does
 };
 
-// One buffer: k and q [TCH, Dp], v [TCH, CP] (CC rounded up to 16 bytes), coefficients [TCH, 12].
+// One buffer: k and q [TCH, Dp], v [TCH, CP] (CC rounded up to 16 bytes), the coefficients.
 __host__ __device__ constexpr int head_v_floats(int CC) { return (CC + 3) / 4 * 4; }
-__host__ __device__ constexpr int head_buf_floats(int TCH, int Dp, int CC) {
-    return TCH * (2 * Dp + head_v_floats(CC) + DH_COEF);
+__host__ __device__ constexpr int head_buf_floats(int TCH, int Dp, int CC, int n) {
+    return TCH * (2 * Dp + head_v_floats(CC) + head_coefs(n));
 }
 
 // grid (column groups, H, B).  A CTA has CC columns of one head of one sequence; L lanes hold
-// NC neighbouring columns, 16 rows of each a lane (L * 16 >= d).  A lane's rows are four quads,
+// NC neighbouring columns, R rows of each a lane (L * R >= d).  A lane's rows are R / 4 quads,
 // quad i of lane l being rows (i L + l) 4 .. + 3: the lanes of a column read consecutive 16
 // bytes of a token's row, the columns of a warp the same ones.  Tokens come TCH at a time
 // through two buffers filled by asynchronous copies; rows beyond a chunk's last token are
 // zeroed where a round reads them.
-template <int L, int NC, int N>
+//
+// A round's 2 N dot products of a column are summed over its lanes so that lane p of every N
+// ends with those of token p (each exchange halves the sums a lane still carries), and, where
+// there are more lanes, with those of some of the columns alone.  That lane forms token p's
+// right-hand side, all lanes take all of them and solve for the writes, and the lane finishes
+// its token's read-out.
+template <int L, int R, int NC, int N>
 __global__ void __launch_bounds__(128)
 head_delta_scan_kernel(HeadScanArgs a, HeadDims dm) {
     pdl_wait();
@@ -194,12 +220,13 @@ head_delta_scan_kernel(HeadScanArgs a, HeadDims dm) {
     if (n <= 0) return;
     const int h = blockIdx.y, grp = h / (dm.H / dm.G);
     const int d = dm.d, dv = dm.dv, C = dm.C(), nq = dm.nq();
-    constexpr int Dp = L * DH_R;
+    constexpr int Dp = L * R;
     const int CC = (int)blockDim.x / L * NC, TCH = a.TCH;
     const int l = threadIdx.x & (L - 1);
     const int jc = (int)(threadIdx.x / L) * NC;              // first of the lane's columns in the CTA
     const int j = blockIdx.x * CC + jc;
-    const int per = head_buf_floats(TCH, Dp, CC), CP = head_v_floats(CC);
+    constexpr int NF = head_coefs(N);
+    const int per = head_buf_floats(TCH, Dp, CC, N), CP = head_v_floats(CC);
     // (padding rows of k and q and columns of v past dv are never copied: zero once)
     for (int i = threadIdx.x; i < 2 * per; i += blockDim.x) smem[i] = 0.f;
     __syncthreads();
@@ -238,31 +265,30 @@ head_delta_scan_kernel(HeadScanArgs a, HeadDims dm) {
                 cp_async_4(sv + tt * CP + c, vrow + (size_t)tt * C + c);
             }
         }
-        const float* crow = a.coef + ((size_t)(t0 + c0) * dm.H + h) * DH_COEF;
-        for (int idx = threadIdx.x; idx < m * (DH_COEF / 4); idx += blockDim.x) {
-            const int tt = idx / (DH_COEF / 4), c4 = (idx - tt * (DH_COEF / 4)) * 4;
-            cp_async_16(sc + tt * DH_COEF + c4, crow + (size_t)tt * dm.H * DH_COEF + c4);
+        const float* crow = a.coef + ((size_t)(t0 + c0) * dm.H + h) * NF;
+        for (int idx = threadIdx.x; idx < m * (NF / 4); idx += blockDim.x) {
+            const int tt = idx / (NF / 4), c4 = (idx - tt * (NF / 4)) * 4;
+            cp_async_16(sc + tt * NF + c4, crow + (size_t)tt * dm.H * NF + c4);
         }
         // places of the last round that no token takes: their k and their numbers are zero
         if (N > 1 && m % N != 0) {
             const int mm = (m + N - 1) / N * N - m;
             for (int idx = threadIdx.x; idx < mm * Dp; idx += blockDim.x) sk[m * Dp + idx] = 0.f;
-            for (int idx = threadIdx.x; idx < mm * DH_COEF; idx += blockDim.x)
-                sc[m * DH_COEF + idx] = 0.f;
+            for (int idx = threadIdx.x; idx < mm * NF; idx += blockDim.x) sc[m * NF + idx] = 0.f;
         }
         cp_async_commit();
     };
 
     fetch(0, smem);
     // S as pairs of rows
-    f32x2 S[NC][DH_R / 2];
+    f32x2 S[NC][R / 2];
     float* srow = a.state + (size_t)slot * a.stride + ((size_t)h * dv + j) * d;
 #pragma unroll
     for (int c = 0; c < NC; ++c) {
         const bool live = j + c < dv;
         const float* s = srow + (size_t)c * d;
 #pragma unroll
-        for (int i = 0; i < DH_R / 4; ++i) {
+        for (int i = 0; i < R / 4; ++i) {
             const int r = (i * L + l) * 4;
             float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
             if (live) {
@@ -295,7 +321,7 @@ head_delta_scan_kernel(HeadScanArgs a, HeadDims dm) {
         __syncthreads();
         for (int tt = 0; tt < m; tt += N) {
             // dot products of the state with the round's k and q
-            f32x2 k2[N][DH_R / 2];
+            f32x2 k2[N][R / 2];
             float ak[NC][N], aq[NC][N];
 #pragma unroll
             for (int i = 0; i < N; ++i) {
@@ -303,7 +329,7 @@ head_delta_scan_kernel(HeadScanArgs a, HeadDims dm) {
 #pragma unroll
                 for (int c = 0; c < NC; ++c) ac[c] = 0ull, rc[c] = 0ull;
 #pragma unroll
-                for (int x = 0; x < DH_R / 4; ++x) {
+                for (int x = 0; x < R / 4; ++x) {
                     const ulonglong2 kv = reinterpret_cast<const ulonglong2*>(sk + (tt + i) * Dp)[x * L];
                     const ulonglong2 qv = reinterpret_cast<const ulonglong2*>(sq + (tt + i) * Dp)[x * L];
                     k2[i][2 * x] = kv.x, k2[i][2 * x + 1] = kv.y;
@@ -324,51 +350,132 @@ head_delta_scan_kernel(HeadScanArgs a, HeadDims dm) {
                     aq[c][i] = lo + hi;
                 }
             }
+            // the sums over a column's lanes, the round's writes, and its read-outs
+            float w[NC][N];
+            const float* cf = sc + tt * NF;                  // numbers of the round
+            if constexpr (L >= N && N > 1) {
+                auto fold = [&](float& keep, float& give, bool up, int bit) {
+                    const float out = up ? keep : give, in = up ? give : keep;
+                    keep = in + __shfl_xor_sync(0xffffffffu, out, bit);
+                };
 #pragma unroll
-            for (int o = 1; o < L; o <<= 1)
+                for (int half = N / 2; half >= 1; half >>= 1)
+#pragma unroll
+                    for (int i = 0; i < half; ++i)
+#pragma unroll
+                        for (int c = 0; c < NC; ++c) {
+                            fold(ak[c][i], ak[c][i + half], l & half, half);
+                            fold(aq[c][i], aq[c][i + half], l & half, half);
+                        }
+                // lanes beyond N: each takes some of the columns, the rest of them sum
+                constexpr int XB = L / N, OWN = NC >= XB ? NC / XB : 1;      // columns a lane ends with
+                int own = 0;                                                 // first of them
+#pragma unroll
+                for (int o = N, half = NC / 2; o < L; o <<= 1, half >>= 1) {
+                    if (half >= 1) {
+                        const bool up = l & o;
+                        if (up) own += half;
+#pragma unroll
+                        for (int c = 0; c < half; ++c) {
+                            fold(ak[c][0], ak[c + half][0], up, o);
+                            fold(aq[c][0], aq[c + half][0], up, o);
+                        }
+                    } else {
+#pragma unroll
+                        for (int c = 0; c < OWN; ++c) {
+                            ak[c][0] += __shfl_xor_sync(0xffffffffu, ak[c][0], o);
+                            aq[c][0] += __shfl_xor_sync(0xffffffffu, aq[c][0], o);
+                        }
+                    }
+                }
+                const int p = l & (N - 1), base = (threadIdx.x & 31) & ~(L - 1);
+                const float* mine = cf + p * NF;
+                const float4 m0 = *reinterpret_cast<const float4*>(mine);
+                float P[N];
+#pragma unroll
+                for (int x = 0; x < N / 4; ++x)
+                    *reinterpret_cast<float4*>(P + 4 * x) =
+                        reinterpret_cast<const float4*>(mine + 4 + N)[x];
+                float rhs[OWN];
+#pragma unroll
+                for (int c = 0; c < OWN; ++c)
+                    rhs[c] = fmaf(-m0.y, ak[c][0], m0.x * sv[(tt + p) * CP + own + c]);
+#pragma unroll
+                for (int c = 0; c < NC; ++c) {
+                    // the lanes that ended with column c: bit N of the lane is the upper half
+                    int who = 0;
+#pragma unroll
+                    for (int o = N, half = NC / 2; o < L && half >= 1; o <<= 1, half >>= 1)
+                        if (c & half) who |= o;
+#pragma unroll
+                    for (int i = 0; i < N; ++i)
+                        w[c][i] = __shfl_sync(0xffffffffu, rhs[c & (OWN - 1)], base | who | i);
+                }
+#pragma unroll
+                for (int i = 1; i < N; ++i) {
+                    float A[N];
+#pragma unroll
+                    for (int x = 0; x < (i + 3) / 4; ++x)
+                        *reinterpret_cast<float4*>(A + 4 * x) =
+                            reinterpret_cast<const float4*>(cf + i * NF + 4)[x];
+#pragma unroll
+                    for (int jj = 0; jj < i; ++jj)
+#pragma unroll
+                        for (int c = 0; c < NC; ++c) w[c][i] = fmaf(-A[jj], w[c][jj], w[c][i]);
+                }
+#pragma unroll
+                for (int c = 0; c < OWN; ++c) {
+                    float o = m0.z * aq[c][0];
+#pragma unroll
+                    for (int jj = 0; jj < N; ++jj) {
+                        float u = w[c][jj];                  // (of column own + c)
+#pragma unroll
+                        for (int e = 1; e < NC / OWN; ++e)
+                            if (own == e * OWN) u = w[e * OWN + c][jj];
+                        o = fmaf(P[jj], u, o);
+                    }
+                    constexpr int TOP = NC >= XB ? L : N * NC;               // lanes that write
+                    if (l < TOP && tt + p < m && j + own + c < dv)
+                        a.out[((size_t)(t0 + c0 + tt + p) * dm.H + h) * dv + j + own + c] = o;
+                }
+            } else {
+#pragma unroll
+                for (int o = 1; o < L; o <<= 1)
+#pragma unroll
+                    for (int i = 0; i < N; ++i)
+#pragma unroll
+                        for (int c = 0; c < NC; ++c) {
+                            ak[c][i] += __shfl_xor_sync(0xffffffffu, ak[c][i], o);
+                            aq[c][i] += __shfl_xor_sync(0xffffffffu, aq[c][i], o);
+                        }
 #pragma unroll
                 for (int i = 0; i < N; ++i)
 #pragma unroll
                     for (int c = 0; c < NC; ++c) {
-                        ak[c][i] += __shfl_xor_sync(0xffffffffu, ak[c][i], o);
-                        aq[c][i] += __shfl_xor_sync(0xffffffffu, aq[c][i], o);
+                        const float* mine = cf + i * NF;
+                        float u = fmaf(-mine[1], ak[c][i], mine[0] * sv[(tt + i) * CP + c]);
+#pragma unroll
+                        for (int jj = 0; jj < i; ++jj) u = fmaf(-mine[4 + jj], w[c][jj], u);
+                        w[c][i] = u;
+                        float o = mine[2] * aq[c][i];
+#pragma unroll
+                        for (int jj = 0; jj <= i; ++jj) o = fmaf(mine[4 + N + jj], w[c][jj], o);
+                        if ((i & (L - 1)) == l && tt + i < m && j + c < dv)
+                            a.out[((size_t)(t0 + c0 + tt + i) * dm.H + h) * dv + j + c] = o;
                     }
-            // the round's writes one after another, and its read-outs
-            float w[NC][N];
-            float total = 1.f;
-#pragma unroll
-            for (int i = 0; i < N; ++i) {
-                const float4* cf = reinterpret_cast<const float4*>(sc + (tt + i) * DH_COEF);
-                const float4 c0v = cf[0], c1v = cf[1], c2v = cf[2];
-                const float A[3] = {c0v.z, c0v.w, c1v.x};
-                const float P[4] = {c1v.z, c1v.w, c2v.x, c2v.y};
-                if (i == 0) total = c2v.w;
-#pragma unroll
-                for (int c = 0; c < NC; ++c) {
-                    float u = fmaf(-c0v.y, ak[c][i], c0v.x * sv[(tt + i) * CP + c]);
-#pragma unroll
-                    for (int jj = 0; jj < 3; ++jj)
-                        if (jj < i) u = fmaf(-A[jj], w[c][jj], u);
-                    w[c][i] = u;
-                    float o = c1v.y * aq[c][i];
-#pragma unroll
-                    for (int jj = 0; jj < 4; ++jj)
-                        if (jj <= i) o = fmaf(P[jj], w[c][jj], o);
-                    if ((i & (L - 1)) == l && tt + i < m && j + c < dv)
-                        a.out[((size_t)(t0 + c0 + tt + i) * dm.H + h) * dv + j + c] = o;
-                }
             }
+            const float total = cf[4 + N - 1];
+            const f32x2 g2 = pack2(total, total);
 #pragma unroll
             for (int c = 0; c < NC; ++c) {
-                const f32x2 g2 = pack2(total, total);
 #pragma unroll
-                for (int x = 0; x < DH_R / 2; ++x) S[c][x] = mul2(S[c][x], g2);
+                for (int x = 0; x < R / 2; ++x) S[c][x] = mul2(S[c][x], g2);
 #pragma unroll
                 for (int i = 0; i < N; ++i) {
-                    const float wu = sc[(tt + i) * DH_COEF + 10] * w[c][i];
+                    const float wu = cf[i * NF + 3] * w[c][i];
                     const f32x2 u2 = pack2(wu, wu);
 #pragma unroll
-                    for (int x = 0; x < DH_R / 2; ++x) S[c][x] = fma2(k2[i][x], u2, S[c][x]);
+                    for (int x = 0; x < R / 2; ++x) S[c][x] = fma2(k2[i][x], u2, S[c][x]);
                 }
             }
         }
@@ -380,7 +487,7 @@ head_delta_scan_kernel(HeadScanArgs a, HeadDims dm) {
         if (j + c >= dv) continue;
         float* s = srow + (size_t)c * d;
 #pragma unroll
-        for (int i = 0; i < DH_R / 4; ++i) {
+        for (int i = 0; i < R / 4; ++i) {
             const int r = (i * L + l) * 4;
             float4 x;
             unpack2(S[c][2 * i], x.x, x.y);
@@ -479,7 +586,7 @@ int check_head_dims(const HeadDims& dm) {
     AGV_REQUIRE(dm.G > 0 && dm.H > 0 && dm.d > 0 && dm.dv > 0, "head_delta: bad sizes");
     AGV_REQUIRE(dm.H % dm.G == 0, "head_delta: %d heads are not a multiple of %d query/key heads",
                 dm.H, dm.G);
-    AGV_REQUIRE(dm.d <= 32 * DH_R, "head_delta: key heads of %d exceed %d", dm.d, 32 * DH_R);
+    AGV_REQUIRE(dm.d <= DH_MAX_D, "head_delta: key heads of %d exceed %d", dm.d, DH_MAX_D);
     return 0;
 }
 
@@ -492,13 +599,29 @@ int head_row(RowIn<float>& in, const float* row, long long ld, const float* part
     return 0;
 }
 
-template <int L, int NC, int N>
-int launch_head_scan(const HeadScanArgs& a, const HeadDims& dm, int B, int threads, size_t smem,
-                     cudaStream_t stream) {
+template <int L, int R, int NC, int N>
+int launch_head_scan(HeadScanArgs a, const HeadDims& dm, int B, cudaStream_t stream) {
+    // 128 threads a CTA where the columns allow, whole warps always
+    int threads = 128;
+    while (threads > 32 && threads / 2 / L * NC >= dm.dv) threads >>= 1;
     const int CC = threads / L * NC;
+    a.TCH = N > 1 ? 16 : 1;
+    while (a.TCH > N && 2 * head_buf_floats(a.TCH, L * R, CC, N) * sizeof(float) > 48 * 1024)
+        a.TCH >>= 1;
+    const size_t smem = 2 * (size_t)head_buf_floats(a.TCH, L * R, CC, N) * sizeof(float);
+    a.vec_v = a.vec_v && CC % 4 == 0;
+    auto kern = head_delta_scan_kernel<L, R, NC, N>;
+    if (smem > 48 * 1024) {
+        static bool configured = false;
+        if (!configured) {
+            AGV_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                             100 * 1024));
+            configured = true;
+        }
+        AGV_REQUIRE(smem <= 100 * 1024, "head_delta_scan: %d bytes of shared memory", (int)smem);
+    }
     // (few CTAs, each a long dependent chain: spread over the SMs)
-    agv_launch_after(head_delta_scan_kernel<L, NC, N>,
-                     dim3((unsigned)((dm.dv + CC - 1) / CC), (unsigned)dm.H, (unsigned)B),
+    agv_launch_after(kern, dim3((unsigned)((dm.dv + CC - 1) / CC), (unsigned)dm.H, (unsigned)B),
                      (unsigned)threads, smem, stream, a, dm);
     AGV_LAUNCH_OK("head_delta_scan_kernel");
     return 0;
@@ -506,31 +629,33 @@ int launch_head_scan(const HeadScanArgs& a, const HeadDims& dm, int B, int threa
 
 }  // namespace
 
-AGV_API int agv_head_delta_coef_numel() { return DH_COEF; }
+// Numbers a token and head (see delta_coef_kernel).
+AGV_API int agv_head_delta_coefs(int several, int d) { return head_coefs(several ? head_round(d) : 1); }
 
 // u: [T, 2 G d + H dv] 32-bit, q | k | v after the convolution; decay: [T, H, 2] 32-bit, the
 // decay first; row / part: the stacked projection [T, W] 32-bit (row stride ld) or [n_splits, T,
 // W] partial sums, whose columns b_off .. b_off + H are beta's logits.  several != 0: sequences
-// may bring more than one token.  coef: [T, H, 12].
+// may bring more than one token.  coef: [T, H, agv_head_delta_coefs(several, d)].
 AGV_API int agv_head_delta_coef(const float* u, const float* decay, const float* row, long long ld,
-                                const float* part, int n_splits, int T, int W, int b_off, int G,
-                                int H, int d, int dv, float eps_unit, float q_mult, int several,
-                                const int* seq_index, const int* cu, float* coef,
-                                cudaStream_t stream) {
+                                const float* part, int n_splits, int T, int W, int b_off, int B,
+                                int G, int H, int d, int dv, float eps_unit, float q_mult,
+                                int several, const int* cu, float* coef, cudaStream_t stream) {
     const HeadDims dm{G, H, d, dv};
     if (int rc = check_head_dims(dm)) return rc;
-    AGV_REQUIRE(T >= 0 && b_off >= 0 && b_off + H <= W, "head_delta_coef: bad sizes");
+    AGV_REQUIRE(T >= 0 && B >= 1 && b_off >= 0 && b_off + H <= W, "head_delta_coef: bad sizes");
     AGV_REQUIRE(agv_aligned(coef, 16), "head_delta_coef: the output must be 16-byte aligned");
     if (T == 0) return 0;
     RowIn<float> in;
     if (int rc = head_row(in, row, ld, part, n_splits, T, W)) return rc;
-    const unsigned grid = (unsigned)(((long long)T * G + 7) / 8);
-    if (several)
-        agv_launch(delta_coef_kernel<DH_ROUND>, grid, 256, 0, stream, u, decay, in, b_off, dm, T,
-                   eps_unit, q_mult, seq_index, cu, coef);
-    else
-        agv_launch(delta_coef_kernel<1>, grid, 256, 0, stream, u, decay, in, b_off, dm, T, eps_unit,
-                   q_mult, seq_index, cu, coef);
+#define AGV_HC(N)                                                                                \
+    agv_launch(delta_coef_kernel<N>,                                                            \
+               (unsigned)(((long long)(T / N + B) * G + DH_COEF_WARPS - 1) / DH_COEF_WARPS),     \
+               DH_COEF_WARPS * 32, 0, stream, u, decay, in, b_off, dm, T, B, eps_unit, q_mult,   \
+               cu, coef)
+    if (!several) AGV_HC(1);
+    else if (head_round(d) == 8) AGV_HC(8);
+    else AGV_HC(4);
+#undef AGV_HC
     AGV_LAUNCH_OK("delta_coef_kernel");
     return 0;
 }
@@ -548,34 +673,35 @@ AGV_API int agv_head_delta_scan(const float* u, const float* coef, float* out, i
     AGV_REQUIRE(B <= 65535 && H <= 65535, "head_delta_scan: batch or head count exceeds the grid limit");
     AGV_REQUIRE(agv_aligned(coef, 16), "head_delta_scan: the coefficients must be 16-byte aligned");
     if (T == 0 || B == 0) return 0;
-    int L = 1;
-    while (L * DH_R < d) L <<= 1;
-    // two columns a lane where the launch still fills the GPU, 128 threads a CTA where the
-    // columns allow, whole warps always
-    const long long lanes = (long long)B * H * dv * L;
-    const int NC = several && L > 1 && lanes >= 148LL * 4 * 32 ? 2 : 1;
-    int threads = 128;
-    while (threads > 32 && threads / 2 / L * NC >= dv) threads >>= 1;
-    const int CC = threads / L * NC, Dp = L * DH_R;
-    int TCH = several ? 16 : 1;
-    while (TCH > DH_ROUND && 2 * head_buf_floats(TCH, Dp, CC) * sizeof(float) > 48 * 1024) TCH >>= 1;
-    const size_t smem = 2 * (size_t)head_buf_floats(TCH, Dp, CC) * sizeof(float);
-    AGV_REQUIRE(smem <= 48 * 1024, "head_delta_scan: key heads of %d need too much shared memory", d);
     const int C = dm.C();
-    HeadScanArgs a{u, coef, out, state, state_stride, slots, cu, TCH, 0, 0, 0};
+    HeadScanArgs a{u, coef, out, state, state_stride, slots, cu, 0, 0, 0, 0};
     a.vec = d % 4 == 0 && C % 4 == 0 && agv_aligned(u, 16);
-    a.vec_v = dv % 4 == 0 && CC % 4 == 0 && C % 4 == 0 && (2 * dm.nq()) % 4 == 0 && agv_aligned(u, 16);
+    a.vec_v = dv % 4 == 0 && C % 4 == 0 && (2 * dm.nq()) % 4 == 0 && agv_aligned(u, 16);
     a.vec_s = d % 4 == 0 && state_stride % 4 == 0 && agv_aligned(state, 16);
-#define AGV_HS(LL)                                                                              \
-    case LL:                                                                                    \
-        if (!several) return launch_head_scan<LL, 1, 1>(a, dm, B, threads, smem, stream);       \
-        if (NC == 2) return launch_head_scan<LL, 2, DH_ROUND>(a, dm, B, threads, smem, stream); \
-        return launch_head_scan<LL, 1, DH_ROUND>(a, dm, B, threads, smem, stream)
-    switch (L) {
-        AGV_HS(1); AGV_HS(2); AGV_HS(4); AGV_HS(8); AGV_HS(16); AGV_HS(32);
+#define AGV_HS(L, R, NC, N) return launch_head_scan<L, R, NC, N>(a, dm, B, stream)
+    if (!several) {
+        if (d <= 16) AGV_HS(1, 16, 1, 1);
+        if (d <= 32) AGV_HS(2, 16, 1, 1);
+        if (d <= 64) AGV_HS(4, 16, 1, 1);
+        if (d <= 128) AGV_HS(8, 16, 1, 1);
+        if (d <= 256) AGV_HS(16, 16, 1, 1);
+        AGV_HS(32, 16, 1, 1);
     }
+    if (d <= 16) AGV_HS(1, 16, 1, 4);
+    if (d <= 32) AGV_HS(4, 8, 1, 4);
+    // (more columns a lane, and so fewer reads of k and q a column, where the launch has more
+    // CTAs than the SMs can take at once anyway)
+    if (d <= 64) {
+        if ((long long)B * H * ((dv + 7) / 8) > 296) AGV_HS(16, 4, 2, 8);
+        AGV_HS(16, 4, 1, 8);
+    }
+    if (d <= 128) {
+        if ((long long)B * H * ((dv + 15) / 16) > 192) AGV_HS(16, 8, 4, 8);
+        AGV_HS(16, 8, 2, 8);
+    }
+    if (d <= 256) AGV_HS(32, 8, 4, 8);
+    AGV_HS(32, 16, 1, 8);
 #undef AGV_HS
-    return agv_fail(-1, "head_delta_scan: %d lanes a column", L);
 }
 
 // o: [T, H * dv] 32-bit; the gate: columns g_off .. g_off + H dv of the stacked projection (row /

@@ -903,7 +903,9 @@ def delta_scan(qkv: torch.Tensor, beta: torch.Tensor, a: torch.Tensor, dt_bias: 
     lib.agv_delta_scan_work.restype = ctypes.c_longlong
     # scratch for what does not depend on the state (k, the decay, their products), per head
     work = ctx.new(int(lib.agv_delta_scan_work(T, n_heads, head_dim)), dtype=torch.float32)
-    with _span("delta_scan", _nbytes(qkv, beta, a, out) + 2 * work.numel() * 4, flops):
+    # (the scratch is not counted: the rule has to read and write its inputs, outputs and state)
+    with _span("delta_scan", _nbytes(qkv, beta, a, out) +
+               8 * ctx.batch * n_heads * head_dim * value_dim, flops):
         _check(lib.agv_delta_scan(_ptr(qkv), _ptr(beta), _ptr(a), _ptr(dt_bias), _ptr(neg_a),
                                   _ptr(out), T, ctx.batch, n_qk_heads, n_heads, head_dim,
                                   value_dim, sp, ss, _ptr(ctx.slots), _ptr(ctx.cu_seqlens),
@@ -925,7 +927,9 @@ def delta_out(o: torch.Tensor, gate: torch.Tensor, w: torch.Tensor, eps: float, 
 
 
 
-HEAD_DELTA_COEF = 12        # numbers a token and head (checked against the library's)
+def head_delta_coefs(ctx, head_dim: int) -> int:
+    """How many numbers ``head_delta_coef`` makes of a token and head in a step of this kind."""
+    return library().agv_head_delta_coefs(0 if ctx.mode == "decode" else 1, head_dim)
 
 
 def head_delta_coef(u: torch.Tensor, decay: torch.Tensor, row: Optional[torch.Tensor],
@@ -935,7 +939,7 @@ def head_delta_coef(u: torch.Tensor, decay: torch.Tensor, row: Optional[torch.Te
     """What the delta rule with a decay per head needs of a token besides its vectors: u [T,
     2 G d + H dv] = q | k | v after the convolution, decay [T, H, 2] (the decay first), beta =
     sigmoid of columns ``b_offset`` .. + H of the stacked projection (32-bit rows [T, W] or
-    ``partial`` [S, T, W]); coef [T, H, 12], see ``csrc/delta_head.cu``."""
+    ``partial`` [S, T, W]); coef [T, H, ``head_delta_coefs``], see ``csrc/delta_head.cu``."""
     T = u.shape[0]
     rp, ld, pp, ns = _f32_row_input(row, partial, T, W)
     for t, n in ((u, "u"), (decay, "decay"), (coef, "coef")):
@@ -943,13 +947,12 @@ def head_delta_coef(u: torch.Tensor, decay: torch.Tensor, row: Optional[torch.Te
     assert u.shape == (T, 2 * n_qk_heads * head_dim + n_heads * value_dim)
     assert decay.shape == (T, n_heads, 2)
     lib = library()
-    assert coef.shape == (T, n_heads, lib.agv_head_delta_coef_numel())
+    assert coef.shape == (T, n_heads, head_delta_coefs(ctx, head_dim))
     with _span("delta_coef", T * 2 * n_qk_heads * head_dim * 4 + _nbytes(decay, coef)):
         _check(lib.agv_head_delta_coef(
-            _ptr(u), _ptr(decay), rp, ld, pp, ns, T, W, b_offset, n_qk_heads, n_heads, head_dim,
-            value_dim, ctypes.c_float(unit_eps), ctypes.c_float(q_mult),
-            0 if ctx.mode == "decode" else 1, _ptr(ctx.seq_index), _ptr(ctx.cu_seqlens),
-            _ptr(coef), _stream()))
+            _ptr(u), _ptr(decay), rp, ld, pp, ns, T, W, b_offset, ctx.batch, n_qk_heads, n_heads,
+            head_dim, value_dim, ctypes.c_float(unit_eps), ctypes.c_float(q_mult),
+            0 if ctx.mode == "decode" else 1, _ptr(ctx.cu_seqlens), _ptr(coef), _stream()))
 
 
 def head_delta_scan(u: torch.Tensor, coef: torch.Tensor, out: torch.Tensor, ctx,
@@ -962,7 +965,8 @@ def head_delta_scan(u: torch.Tensor, coef: torch.Tensor, out: torch.Tensor, ctx,
     for t, n in ((u, "u"), (coef, "coef"), (out, "out")):
         _f32(t, n); _dense(t, n)
     assert u.shape == (T, 2 * n_qk_heads * head_dim + n_heads * value_dim)
-    assert out.shape == (T, n_heads * value_dim) and coef.shape[:2] == (T, n_heads)
+    assert out.shape == (T, n_heads * value_dim)
+    assert coef.shape == (T, n_heads, head_delta_coefs(ctx, head_dim))
     sp, ss = _state_args(state)
     with _span("delta_scan", _nbytes(u, coef, out) +
                8 * ctx.batch * n_heads * head_dim * value_dim,

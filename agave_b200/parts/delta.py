@@ -218,7 +218,7 @@ class HeadDeltaMixer:
         kernels.ssm_conv(row, part, T, W, 0, s.conv_taps, self.conv_w, None, u, None, state,
                          self.state_numel, ctx, dt_offset=C, dt_bias=self.dt_bias,
                          neg_a=self.neg_a, coef=decay)
-        coef = ctx.new(T, H, kernels.HEAD_DELTA_COEF, dtype=f32)
+        coef = ctx.new(T, H, kernels.head_delta_coefs(ctx, d), dtype=f32)
         kernels.head_delta_coef(u, decay, row, part, W, C + H, G, H, d, dv, s.unit_eps,
                                 float(d) ** -0.5, ctx, coef)
         o = ctx.new(T, self.n_v, dtype=f32)

@@ -45,7 +45,11 @@ decoder of equal width, heads, head size, experts, layers and vocabulary.  ``--c
 sets the Savovik decoder (both branches of a layer from one norm with a gate each; chunked
 attention beside a selective scan, the head-wise state-space scan, windowed attention with
 capped scores) beside a Kadavik decoder of equal width, heads, head size, layers and vocabulary
-with dense feed-forwards of equal weight.
+with dense feed-forwards of equal weight.  ``--compare pubunex`` sets the Pubunex decoder (the
+delta rule with one decay per head, attention with biases, latent attention with a sink; experts
+whose weight multiplies their input beside a shared one; both branches from one norm; layers that
+run twice) beside a Bovozen decoder of equal width, heads, head size, experts, layer runs and
+vocabulary.
 """
 import argparse
 import json
@@ -395,7 +399,38 @@ def compare_configs_savovik(size):
     return savovik, kadavik
 
 
-COMPARE_BUILDERS = {"savovik": (compare_configs_savovik, "kadavik"),
+def compare_configs_pubunex(size):
+    """Pubunex beside Bovozen, the library's other decoder with the delta rule and routed experts
+    beside a shared one: equal width, heads, head size, experts, layer runs and vocabulary.
+    Pubunex's layers are the delta rule (as many heads and taps, a decay per head), attention
+    with biases (half the head rotated, scaled frequencies) and latent attention (the sizes of
+    the Zazerax comparison); some of them run twice, so that there are as many layer runs as
+    Bovozen has layers, with fewer weights."""
+    H, A, G, d, E, top, ff, groups, keep, L, V = COMPARE_SIZES[size]
+    z = ZAZERAX_SIZES[size]
+    att = {"dim": d, "heads": A, "kv_heads": G,
+           "rot": {"base": 1000000.0, "dims": d // 2,
+                   "scaling": {"factor": 8.0, "fast": 32.0, "original": 8192, "slow": 1.0}},
+           "scale": d ** -0.5, "vdim": d}
+    lat = {"dim": z["d"], "heads": A, "kv_rank": z["R"],
+           "rot": {"base": 1000000.0, "dims": z["r"]}, "rot_dim": z["r"],
+           "scale": (z["d"] + z["r"]) ** -0.5, "vdim": z["dv"]}
+    rec = {"conv": 4, "dim": d, "heads": A, "kv_heads": G, "vdim": d}
+    mlp = {"expert": {"ff": ff, "limit": 7.0}, "kind": "moe", "router": {"experts": E, "top": top},
+           "shared": {"ff": 2 * ff, "limit": 7.0}}
+    delta, attention, latent = ("delta", rec), ("attention", att), ("latent_attention", lat)
+    kinds, stop = (([delta, attention, delta, latent], 4) if L == 8 else
+                   ([delta, attention, latent], 1))
+    layers = [{"mixer": m, "mlp": mlp, "type": k} for k, m in kinds]
+    assert len(layers) + stop == L
+    pubunex = {"architecture": "Pubunex", "layers": layers,
+               "loop": {"start": 0, "stop": stop, "times": 2}, "norm": {"eps": 1e-6}, "vocab": V,
+               "width": H}
+    return pubunex, compare_configs_bovozen(size)[0]
+
+
+COMPARE_BUILDERS = {"pubunex": (compare_configs_pubunex, "bovozen"),
+                    "savovik": (compare_configs_savovik, "kadavik"),
                     "ramilorn": (compare_configs, "gemma3"),
                     "kadavik": (compare_configs_kadavik, "bovozen"),
                     "zazerax": (compare_configs_zazerax, "gemma3"),
