@@ -71,8 +71,11 @@ __device__ __forceinline__ float gelu_tanh_fast(float t) {
     return 0.5f * t * (1.0f + th);
 }
 __device__ __forceinline__ float silu_fast(float t) { return __fdividef(t, 1.0f + __expf(-t)); }
+// (the bounded gate is an instantiation of its own: the others' epilogues stay as short as they
+// are, which a decode step's kernels, each a few microseconds from a cold instruction cache, feel)
+template <bool BOUNDED>
 __device__ __forceinline__ float gated_fast(float g, float u, const GateAct& act) {
-    if (act.kind == AGV_ACT_CLAMPED) return clamped_gate_fast(g, u, act);
+    if constexpr (BOUNDED) return clamped_gate_fast(g, u, act);
     return (act.kind == AGV_ACT_SILU ? silu_fast(g) : gelu_tanh_fast(g)) * u;
 }
 // The activation a plain product may carry: 2 the squared relu, 3 the erf GELU.
@@ -129,7 +132,7 @@ template <> __device__ __forceinline__ void store_out<__nv_bfloat16>(__nv_bfloat
     *p = __float2bfloat16_rn(v);
 }
 
-template <int BN, int MODE, typename TO, int SLIM = 0>
+template <int BN, int MODE, typename TO, int SLIM = 0, bool BOUNDED = false>
 __global__ void __launch_bounds__(GEMM_THREADS, 1)
 gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_w,
                     const __grid_constant__ CUtensorMap map_w2,
@@ -345,7 +348,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_w,
                             if (n < T) {
                                 const float gv = __uint_as_float(r[j]);
                                 const float uv = xchg[(c + j) * 64 + quarter * 32 + lane];
-                                store_out<TO>(obase + (size_t)n * ldc + f, gated_fast(gv, uv, act));
+                                store_out<TO>(obase + (size_t)n * ldc + f, gated_fast<BOUNDED>(gv, uv, act));
                             }
                         }
                     }
@@ -369,7 +372,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_w,
                     for (int j = 0; j < 16; ++j) {
                         float v = __uint_as_float(r[j]);
                         if (GATED)
-                            v = gated_fast(v, __uint_as_float(u[j]), act);
+                            v = gated_fast<BOUNDED>(v, __uint_as_float(u[j]), act);
                         else if (MODE == 0 && act.kind >= 2) v = plain_act(v, act.kind);
                         store_out<TO>(ctile + (c + j) * TILE_M + fl, v);
                     }
@@ -453,7 +456,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_w,
                         acc += inbox[((size_t)q * BN + n) * rows + jl];
                         if (HALF) up += inbox[((size_t)q * BN + n) * rows + per + jl];
                     }
-                    if (HALF) acc = gated_fast(acc, up, act);
+                    if (HALF) acc = gated_fast<BOUNDED>(acc, up, act);
                     else if (MODE == 0 && act.kind >= 2) acc = plain_act(acc, act.kind);
                     store_out<TO>(gout + (size_t)(n0 + n) * ldc + m0 + fl, acc);
                 }
@@ -480,7 +483,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_w,
                         float up = 0.f;
 #pragma unroll
                         for (int q = 0; q < 8; ++q) up += pu[q];
-                        acc = gated_fast(acc, up, act);
+                        acc = gated_fast<BOUNDED>(acc, up, act);
                     } else if (MODE == 0 && act.kind >= 2) {
                         acc = plain_act(acc, act.kind);
                     }
@@ -709,7 +712,7 @@ __device__ __forceinline__ void qkv_epilogue(uint32_t lane_base, int m0, int tok
     }
 }
 
-template <int BN, int MODE, typename TO>
+template <int BN, int MODE, typename TO, bool BOUNDED = false>
 __global__ void __launch_bounds__(PERSISTENT_THREADS, 1)
 gemm_tcgen05_persistent_kernel(const __grid_constant__ CUtensorMap map_w,
                                const __grid_constant__ CUtensorMap map_w2,
@@ -897,7 +900,7 @@ gemm_tcgen05_persistent_kernel(const __grid_constant__ CUtensorMap map_w,
             auto work = [&](const uint32_t (&r)[16], const uint32_t (&u)[16], int c) {
                 if constexpr (GATED) {
                     float v[16];
-                    if (act.kind == AGV_ACT_CLAMPED) {
+                    if constexpr (BOUNDED) {
 #pragma unroll
                         for (int j = 0; j < 16; ++j)
                             v[j] = clamped_gate_fast(__uint_as_float(r[j]), __uint_as_float(u[j]),
@@ -929,12 +932,7 @@ gemm_tcgen05_persistent_kernel(const __grid_constant__ CUtensorMap map_w,
                     }
                     return;
                 }
-                if (GATED) {
-#pragma unroll
-                    for (int j = 0; j < 16; ++j)
-                        store_out<TO>(wst + j * 32 + lane,
-                                      gated_fast(__uint_as_float(r[j]), __uint_as_float(u[j]), act));
-                } else if (MODE == 0 && act.kind >= 2) {
+                if (MODE == 0 && act.kind >= 2) {
                     // plain product with an activation on it
 #pragma unroll
                     for (int j = 0; j < 16; ++j)
@@ -1068,6 +1066,7 @@ __device__ __forceinline__ void mbar_arrive_cluster(uint32_t bar_cluster_addr) {
                  : "memory");
 }
 
+template <bool BOUNDED>
 __global__ void __launch_bounds__(PERSISTENT_THREADS, 1)
 gemm_tcgen05_pair_gated_kernel(const __grid_constant__ CUtensorMap map_w,
                                const __grid_constant__ CUtensorMap map_w2,
@@ -1225,7 +1224,7 @@ gemm_tcgen05_pair_gated_kernel(const __grid_constant__ CUtensorMap map_w,
             };
             auto work = [&](const uint32_t (&r)[16], const uint32_t (&u)[16], int c) {
                 float v[16];
-                if (act.kind == AGV_ACT_CLAMPED) {
+                if constexpr (BOUNDED) {
 #pragma unroll
                     for (int j = 0; j < 16; ++j)
                         v[j] = clamped_gate_fast(__uint_as_float(r[j]), __uint_as_float(u[j]), act);
@@ -1324,16 +1323,21 @@ int make_map(CUtensorMap* out, const void* ptr, long long rows, long long K, lon
     return 0;
 }
 
-template <int BN, int MODE, typename TO, int SLIM = 0>
+template <int BN, int MODE, typename TO, int SLIM = 0, bool BOUNDED = false>
 int launch(const CUtensorMap& mw, const CUtensorMap& mw2, const CUtensorMap& mx, void* out, int T,
            int N, int K, long long ldc, long long split_stride, int splits, int kb_per_split,
            GateAct act, int cluster_reduce, cudaStream_t stream, int* argmax_out = nullptr) {
+    if constexpr (MODE != 0 && !BOUNDED)
+        if (act.kind == AGV_ACT_CLAMPED)
+            return launch<BN, MODE, TO, SLIM, true>(mw, mw2, mx, out, T, N, K, ldc, split_stride,
+                                                    splits, kb_per_split, act, cluster_reduce,
+                                                    stream, argmax_out);
     using TL = Tile<BN, MODE, SLIM>;
     static_assert(MODE != 0 || BN * RED_LD * 4 <= TL::STAGES * TL::STAGE_BYTES,
                   "a partial tile must fit the ring of stages");
     AGV_REQUIRE(!cluster_reduce || BN * RED_LD * 4 <= TL::STAGES * TL::STAGE_BYTES,
                 "linear: a partial tile of %d tokens does not fit the ring of stages", BN);
-    auto kern = gemm_tcgen05_kernel<BN, MODE, TO, SLIM>;
+    auto kern = gemm_tcgen05_kernel<BN, MODE, TO, SLIM, BOUNDED>;
     static bool configured = false;
     if (!configured) {
         AGV_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize,
@@ -1355,13 +1359,18 @@ int launch(const CUtensorMap& mw, const CUtensorMap& mw2, const CUtensorMap& mx,
     return 0;
 }
 
-template <int BN, int MODE, typename TO>
+template <int BN, int MODE, typename TO, bool BOUNDED = false>
 int launch_persistent(const CUtensorMap& mw, const CUtensorMap& mw2, const CUtensorMap& mx,
                       void* out, int T, int N, int K, long long ldc, long long split_stride,
                       int splits, int kb_per_split, GateAct act, cudaStream_t stream,
                       const QkvEpilogue& qe = QkvEpilogue{}) {
+    if constexpr (MODE == 1 && !BOUNDED)
+        if (act.kind == AGV_ACT_CLAMPED)
+            return launch_persistent<BN, MODE, TO, true>(mw, mw2, mx, out, T, N, K, ldc,
+                                                         split_stride, splits, kb_per_split, act,
+                                                         stream, qe);
     using TL = PTile<BN, MODE>;
-    auto kern = gemm_tcgen05_persistent_kernel<BN, MODE, TO>;
+    auto kern = gemm_tcgen05_persistent_kernel<BN, MODE, TO, BOUNDED>;
     static bool configured = false;
     static int sms = 0;
     if (!configured) {
@@ -1382,9 +1391,10 @@ int launch_persistent(const CUtensorMap& mw, const CUtensorMap& mw2, const CUten
     return 0;
 }
 
+template <bool BOUNDED>
 int launch_pair_gated(const CUtensorMap& mw, const CUtensorMap& mw2, const CUtensorMap& mx,
                       void* out, int T, int N, int K, long long ldc, GateAct act, cudaStream_t stream) {
-    auto kern = gemm_tcgen05_pair_gated_kernel;
+    auto kern = gemm_tcgen05_pair_gated_kernel<BOUNDED>;
     static bool configured = false;
     static int sms = 0;
     if (!configured) {
@@ -1526,7 +1536,9 @@ AGV_API int agv_linear_tc(const void* x, const void* w, const void* w2, void* ou
             static const bool pairs = getenv("AGAVE_B200_CTA_PAIRS") == nullptr ||
                                       getenv("AGAVE_B200_CTA_PAIRS")[0] != '0';
             if (pairs && T >= 2 * TILE_M)
-                return launch_pair_gated(mw, mw2, mx, out, T, N, K, ldc, act, stream);
+                return act_kind == AGV_ACT_CLAMPED
+                           ? launch_pair_gated<true>(mw, mw2, mx, out, T, N, K, ldc, act, stream)
+                           : launch_pair_gated<false>(mw, mw2, mx, out, T, N, K, ldc, act, stream);
             return launch_persistent<128, 1, __nv_bfloat16>(mw, mw2, mx, out, T, N, K, ldc, 0, 1,
                                                             kb_total, act, stream);
         }

@@ -193,17 +193,27 @@ moe_grouped_tc_kernel(const __grid_constant__ CUtensorMap map_w,
                 tc_ld16(lane_base + c, r);
                 if (GATED) tc_ld16(lane_base + MT_N + c, u);
                 tc_wait_ld();
+                if constexpr (GATED) {
+                    auto emit = [&](auto gate) {
 #pragma unroll
-                for (int j = 0; j < 16; ++j) {
-                    float v = __uint_as_float(r[j]);
-                    if constexpr (GATED) {
-                        float w = __uint_as_float(u[j]);
-                        if (c_scale) v *= s_scale[c + j], w *= s_scale[c + j];
-                        v = mt_act(v, w, act);
-                        ctile[(c + j) * MT_M + fl] = __float2bfloat16_rn(v);
-                    } else {
-                        ctile[(c + j) * MT_M + fl] = v * s_scale[c + j];
-                    }
+                        for (int j = 0; j < 16; ++j)
+                            ctile[(c + j) * MT_M + fl] = __float2bfloat16_rn(
+                                gate(__uint_as_float(r[j]), __uint_as_float(u[j]), c + j));
+                    };
+                    if (c_scale)
+                        emit([&](float g, float w, int n) {
+                            return mt_act(g * s_scale[n], w * s_scale[n], act);
+                        });
+                    else if (act.kind == AGV_ACT_SILU)
+                        emit([](float g, float w, int) {
+                            return __fdividef(g, 1.0f + __expf(-g)) * w;
+                        });
+                    else
+                        emit([&](float g, float w, int) { return mt_act(g, w, act); });
+                } else {
+#pragma unroll
+                    for (int j = 0; j < 16; ++j)
+                        ctile[(c + j) * MT_M + fl] = __uint_as_float(r[j]) * s_scale[c + j];
                 }
             }
         }
