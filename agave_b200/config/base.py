@@ -520,9 +520,9 @@ def default_schedule(n_blocks: int) -> Tuple[LayerCall, ...]:
 
 def looped_schedule(n_blocks: int, start: int, stop: int, times: int,
                     add_embedding: bool = True) -> Tuple[LayerCall, ...]:
-    """Blocks start .. stop-1 run ``times`` times in a row, the others once; every call has a
-    cache entry of its own.  ``add_embedding``: each pass but the first begins with the stream
-    as it was before the first block added."""
+    """A run order in which a stretch of blocks (from ``start`` up to ``stop``, which is not part
+    of it) is gone through ``times`` times and every other block once; every call has a cache
+    entry of its own.  ``add_embedding``: see ``LayerCall``, for every return to ``start``."""
     order = [(i, False) for i in range(start)]
     for t in range(times):
         order += [(i, add_embedding and t > 0 and i == start) for i in range(start, stop)]
