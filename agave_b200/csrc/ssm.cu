@@ -126,6 +126,43 @@ ssm_conv_kernel(RowIn<float> in, int n_tokens, int off, int C, StepArgs st,
     }
 }
 
+// The same for more taps than the forms above hold in registers: a thread has one channel of one
+// token and reads its inputs where they lie.
+template <typename T>
+__global__ void __launch_bounds__(128)
+ssm_conv_long_kernel(RowIn<float> in, int off, int C, int taps, StepArgs st,
+                     const float* __restrict__ w, const float* __restrict__ bias,
+                     float* __restrict__ out, T* __restrict__ rounded, int dt_off, int n_dt,
+                     const float* __restrict__ dt_bias, const float* __restrict__ neg_a,
+                     float* __restrict__ coef) {
+    pdl_wait();
+    pdl_launch_next();
+    const int c = blockIdx.x * 128 + threadIdx.x, t = blockIdx.y, ring_rows = taps - 1;
+    if (c >= C + n_dt) return;
+    if (c >= C) {
+        const int h = c - C;
+        const float dt = softplus_f(in.at(t, dt_off + h) + dt_bias[h]);
+        coef[((size_t)t * n_dt + h) * 2] = expf(neg_a[h] * dt);
+        coef[((size_t)t * n_dt + h) * 2 + 1] = dt;
+        return;
+    }
+    const int e = st.seq_index[t], p = st.positions[t], before = t - st.cu[e], slot = st.slots[e];
+    float* ring = slot >= 0 ? st.state + (size_t)slot * st.stride + st.off + c : nullptr;
+    const float* wc = w + (size_t)c * taps;
+    float acc = bias ? bias[c] : 0.f;
+    for (int k = min(ring_rows, p); k >= 1; --k) {             // oldest input first
+        float x = 0.f;
+        if (k <= before) x = in.at(t - k, off + c);
+        else if (ring) x = ring[(size_t)((p - k) % ring_rows) * C];
+        acc = fmaf(wc[ring_rows - k], x, acc);
+    }
+    const float cur = in.at(t, off + c);
+    const float y = silu_f(fmaf(wc[ring_rows], cur, acc));
+    out[(size_t)t * C + c] = y;
+    if (rounded) rounded[(size_t)t * C + c] = from_f32<T>(y);
+    if (ring && p >= st.lens[e] - ring_rows) ring[(size_t)(p % ring_rows) * C] = cur;
+}
+
 // ---------------------------------------------------------- selective scan
 __host__ __device__ inline int ss_pad(int N) { return N <= 4 ? 4 : N <= 8 ? 8 : N <= 16 ? 16
                                                     : N <= 32 ? 32 : N <= 64 ? 64
@@ -419,7 +456,7 @@ int row_of(RowIn<float>& in, const float* row, long long ld, const float* part, 
     return 0;
 }
 
-constexpr int SSM_MAX_TAPS = 8;
+constexpr int SSM_TAPS = 8;          // taps held in registers; more are read where they lie
 
 template <typename T, int TAPS>
 void launch_conv(const RowIn<float>& in, int n_tokens, int off, int C, const StepArgs& st,
@@ -467,9 +504,9 @@ AGV_API int agv_ssm_conv(const float* row, long long ld, const float* part, int 
     AGV_REQUIRE(T >= 0 && off >= 0 && C > 0 && off + C <= W && n_dt >= 0, "ssm_conv: bad sizes");
     AGV_REQUIRE(n_dt == 0 || (dt_off >= 0 && dt_off + n_dt <= W && dt_bias && neg_a && coef),
                 "ssm_conv: step sizes need their columns, bias, decay and output");
-    AGV_REQUIRE(taps >= 1 && taps <= SSM_MAX_TAPS, "ssm_conv: %d taps, at most %d", taps,
-                SSM_MAX_TAPS);
-    AGV_REQUIRE(T <= 65535 * 8, "ssm_conv: %d tokens exceed the grid limit", T);
+    AGV_REQUIRE(taps >= 1, "ssm_conv: %d taps", taps);
+    AGV_REQUIRE(T <= (taps <= SSM_TAPS ? 65535 * 8 : 65535), "ssm_conv: %d tokens exceed the grid "
+                "limit", T);
     AGV_REQUIRE(taps == 1 || (state && state_stride >= state_off + (long long)(taps - 1) * C),
                 "ssm_conv: the state has no room for the convolution's inputs");
     if (T == 0) return 0;
@@ -480,7 +517,11 @@ AGV_API int agv_ssm_conv(const float* row, long long ld, const float* part, int 
     case K: launch_conv<TT, K>(in, T, off, C, st, conv_w, conv_b, out, (TT*)rounded, dt_off, n_dt, \
                                dt_bias, neg_a, coef, stream); break
 #define AGV_CONVS(TT)                                                                            \
-    switch (taps) {                                                                              \
+    if (taps > SSM_TAPS)                                                                         \
+        agv_launch(ssm_conv_long_kernel<TT>, dim3((unsigned)((C + n_dt + 127) / 128), (unsigned)T), \
+                   128, 0, stream, in, off, C, taps, st, conv_w, conv_b, out, (TT*)rounded, dt_off, \
+                   n_dt, dt_bias, neg_a, coef);                                                  \
+    else switch (taps) {                                                                         \
         AGV_CONV(TT, 1); AGV_CONV(TT, 2); AGV_CONV(TT, 3); AGV_CONV(TT, 4);                      \
         AGV_CONV(TT, 5); AGV_CONV(TT, 6); AGV_CONV(TT, 7); AGV_CONV(TT, 8);                      \
     }

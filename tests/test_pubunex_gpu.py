@@ -265,7 +265,9 @@ def _delta(*a):
 
 DELTA = [(72, _delta(4, 2, 10, 14, 3)), (128, _delta(4, 2, 64, 64, 4)), (96, _delta(1, 1, 16, 16, 1)),
          (76, _delta(2, 1, 130, 33, 6)), (64, _delta(6, 1, 18, 7, 2)), (64, _delta(2, 2, 128, 64, 4)),
-         (48, _delta(3, 3, 1, 1, 4)), (64, _delta(2, 1, 300, 20, 2)), (64, _delta(4, 4, 33, 40, 8)),
+         (48, _delta(3, 3, 1, 1, 4)), (64, _delta(2, 1, 300, 20, 2)),
+         # (more taps than the convolution holds in registers)
+         (64, _delta(2, 1, 24, 20, 9)), (48, _delta(4, 2, 64, 32, 17)), (64, _delta(4, 4, 33, 40, 8)),
          (40, _delta(1, 1, 200, 3, 2)), (64, _delta(12, 3, 128, 128, 2)), (64, _delta(16, 4, 48, 136, 3)),
          # (enough columns for the forms that hold more of them a lane, the last ones partly empty)
          (48, _delta(26, 13, 100, 122, 2)), (48, _delta(40, 5, 40, 61, 2)), (32, _delta(3, 1, 256, 250, 2))]
@@ -300,7 +302,8 @@ def test_every_length_round_a_round_of_the_scan(n):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("m", [_delta(4, 2, 24, 40, 4), _delta(4, 1, 64, 32, 3), _delta(2, 2, 128, 48, 2)])
+@pytest.mark.parametrize("m", [_delta(4, 2, 24, 40, 4), _delta(4, 1, 64, 32, 3), _delta(2, 2, 128, 48, 2),
+                               _delta(2, 2, 16, 24, 12)])
 def test_delta_unequal_batches_and_slots_used_again(dtype, m):
     """A freed slot's state and stored convolution inputs must start at zero again; sequences
     whose rounds begin at any place of the step's tokens."""
